@@ -83,6 +83,12 @@ int mixers_state_space_scan(int dtype, const void* conv, int B, int S, int group
 int mixers_gated_linear_attention(int dtype, const void* proj, int B, int S, int ld, int heads, int dim, int vdim, const void* z,
                                   float tau, float* state, int slot0, const int32_t* pad, float* o, mixers_stream_t stream);
 
+/* Linear attention with one constant decay per head (decay: float [heads]).  proj [B, S, ld]: q | k (heads x dim each) | v (heads x
+ * vdim) from column off, silu applied to all three here when act_silu.  Per head:  M <- decay M + k v^T;  o = M^T q. */
+int mixers_constant_decay_attention(int dtype, const void* proj, int B, int S, int ld, int off, int heads, int dim, int vdim,
+                                    const float* decay, int act_silu, float* state, int slot0, const int32_t* pad, float* o,
+                                    mixers_stream_t stream);
+
 /* out[n, out_col + h * vdim + c] = out_scale * o[n, h, c] / rms(o[n, h, :]) * w[h * w_head_stride + c] * silu(gate[n, off_g + h * vdim + c])
  * (w_head_stride 0: one weight vector [vdim] for every head; vdim: a vector per head, [heads * vdim]).  gate_mode bit 0: the gate
  * is sigmoid(.) instead of silu(.); bit 1: the gate multiplies before the norm, i.e. rms is taken of o * gate. */
@@ -90,9 +96,9 @@ int mixers_gated_rms_norm(int dtype, const float* o, long n_rows, int heads, int
                           const void* w, int w_head_stride, float eps, void* out, int ld_out, int out_col, float out_scale,
                           int gate_mode, mixers_stream_t stream);
 
-/* o[n, c] *= sigmoid(gate[n, off_g + c / per_gate]) in place, o dtype [n_rows, cols] */
-int mixers_sigmoid_gate(int dtype, void* o, long n_rows, int cols, const void* gate, int ld_gate, int off_g, int per_gate,
-                        mixers_stream_t stream);
+/* o[n, c] *= out_scale * sigmoid(gate[n, off_g + c / per_gate]) in place, o dtype: n_rows rows of cols channels, ld_o apart */
+int mixers_sigmoid_gate(int dtype, void* o, long ld_o, long n_rows, int cols, const void* gate, int ld_gate, int off_g, int per_gate,
+                        float out_scale, mixers_stream_t stream);
 
 /* out float [n_rows, width] = scale * (a / rms(a) * w_a + b / rms(b) * w_b): two branch outputs meet as normalised vectors */
 int mixers_rms_pair_sum(int dtype, const void* a, const void* b, const void* w_a, const void* w_b, float eps, float scale, long n_rows,
@@ -102,10 +108,13 @@ int mixers_rms_pair_sum(int dtype, const void* a, const void* b, const void* w_a
  * [n_rows, width], in place):  x += y_a + y_c + y_b + y_d (dtype, dtype, float, float; each may be null);  with pre_gain:
  * x <- x / rms(x) * pre_gain[0] (the norm behind an embedding);  with stack (float [streams, n_rows, width]): the new x is kept
  * as stream `index` and, with coef (dtype [index + 1]), replaced by sum_j coef[j] * stack[j];  h1 = x / rms(x) * gain1[0],
- * h2 = x / rms(x) * gain2[0] in dtype (either may be null). */
+ * h2 = x / rms(x) * gain2[0] in dtype (either may be null).  gain_vectors != 0: gain1 and gain2 are weight vectors [width].
+ * replace != 0: x is replaced by the sum of the addends instead of added to (a stream projected anew).  vec (dtype [width], may be
+ * null) belongs to the sum.  xc (may be null): the new x in dtype, row n at xc + n * ld_xc. */
 int mixers_sum_residual_norms(int dtype, float* x, long n_rows, int width, const void* y_a, const void* y_c, const float* y_b,
                               const float* y_d, const void* pre_gain, float eps, float* stack, long stack_stride, int index,
-                              const void* coef, const void* gain1, const void* gain2, void* h1, void* h2, mixers_stream_t stream);
+                              const void* coef, const void* gain1, const void* gain2, int gain_vectors, void* h1, void* h2, int replace,
+                              const void* vec, void* xc, long ld_xc, mixers_stream_t stream);
 
 /* out = exact (erf) gelu of in, n elements */
 int mixers_gelu_erf(int dtype, const void* in, long n, void* out, mixers_stream_t stream);
@@ -191,12 +200,14 @@ int mixers_wide_qkv_prepare(int dtype, const void* proj, int B, int S, int ld, i
  * channels from off_q, `kv_heads` key heads of k_dim channels from off_k and, if vdim > 0, `kv_heads` value heads from off_v.
  * Inside a head channel rot_off + i pairs with rot_off + i + rot_dims / 2: (u, v) -> (u cos a - v sin a, v cos a + u sin a) * amp,
  * a = position * inv_freq[i] (doubles; angle, sine and cosine in double precision).  k_norm_w (may be null): the first
- * k_norm_cols channels of a key head are divided by their root mean square (eps) and multiplied by k_norm_w first.  q_out dtype
+ * k_norm_cols channels of a key head are divided by their root mean square (eps) and multiplied by k_norm_w first.  unit_rms != 0:
+ * behind the rotation every query and key head is divided by its root mean square over its channels (eps, no weight); values
+ * pass as they are and may be the key columns themselves (off_v = off_k).  q_out dtype
  * [B * S, heads * q_dim]; key of row b, storage index j, head g at k_store + b * k_bs + j * k_ps + g * k_hs (values alike);
  * the new tokens go to index held + t; padding slots store zeros.  dyn as in mixers_window_qk_prepare. */
 int mixers_rope_qk_prepare(int dtype, const void* proj, int B, int S, int ld, int off_q, int off_k, int off_v, int heads, int kv_heads,
                            int q_dim, int k_dim, int vdim, int q_rot_off, int k_rot_off, int rot_dims, const double* inv_freq, float amp,
-                           const void* k_norm_w, int k_norm_cols, float eps, void* q_out, void* k_store, long k_bs, long k_ps, long k_hs,
+                           const void* k_norm_w, int k_norm_cols, float eps, int unit_rms, void* q_out, void* k_store, long k_bs, long k_ps, long k_hs,
                            void* v_store, long v_bs, long v_ps, long v_hs, int held, int shift, const int32_t* pad, const int32_t* dyn,
                            mixers_stream_t stream);
 

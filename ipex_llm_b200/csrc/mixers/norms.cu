@@ -177,15 +177,17 @@ __global__ void gated_rms_norm_wide_kernel(const float* __restrict__ o, int head
     }
 }
 
-// o[n, c] *= sigmoid(gate[n, off_g + c / per_gate]) in place: a gate per channel (per_gate 1) or one per head (per_gate = the
-// head's channels)
+// o[n, c] *= out_scale * sigmoid(gate[n, off_g + c / per_gate]) in place (o: rows of `cols` channels, ld_o apart): a gate per channel
+// (per_gate 1) or one per head (per_gate = the head's channels)
 template <typename T>
-__global__ void sigmoid_gate_kernel(T* __restrict__ o, long n_rows, int cols, const T* __restrict__ gate, int ld_gate, int off_g, int per_gate) {
+__global__ void sigmoid_gate_kernel(T* __restrict__ o, long ld_o, long n_rows, int cols, const T* __restrict__ gate, int ld_gate, int off_g,
+                                    int per_gate, float out_scale) {
     const long total = n_rows * cols;
     for (long i = blockIdx.x * (long)blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
         const long n = i / cols;
         const int c = (int)(i - n * cols);
-        o[i] = from_f<T>(to_f(o[i]) * sigmoid_f(to_f(gate[n * ld_gate + off_g + c / per_gate])));
+        T& e = o[n * ld_o + c];
+        e = from_f<T>(to_f(e) * out_scale * sigmoid_f(to_f(gate[n * ld_gate + off_g + c / per_gate])));
     }
 }
 
@@ -317,12 +319,13 @@ extern "C" int mixers_soft_cap(int dtype, const void* x, long n, float cap, floa
     return mixers_status();
 }
 
-extern "C" int mixers_sigmoid_gate(int dtype, void* o, long n_rows, int cols, const void* gate, int ld_gate, int off_g, int per_gate,
-                                   mixers_stream_t stream) {
+extern "C" int mixers_sigmoid_gate(int dtype, void* o, long ld_o, long n_rows, int cols, const void* gate, int ld_gate, int off_g, int per_gate,
+                                   float out_scale, mixers_stream_t stream) {
     if (n_rows <= 0 || cols <= 0) return 0;
-    if (per_gate < 1) return (int)cudaErrorInvalidValue;
-    MIXERS_DISPATCH(dtype, sigmoid_gate_kernel<T><<<grid_for(n_rows * cols, 256), 256, 0, (cudaStream_t)stream>>>((T*)o, n_rows, cols, (const T*)gate,
-                                                                                                                 ld_gate, off_g, per_gate));
+    if (per_gate < 1 || ld_o < cols) return (int)cudaErrorInvalidValue;
+    MIXERS_DISPATCH(dtype, sigmoid_gate_kernel<T><<<grid_for(n_rows * cols, 256), 256, 0, (cudaStream_t)stream>>>((T*)o, ld_o, n_rows, cols,
+                                                                                                                 (const T*)gate, ld_gate, off_g, per_gate,
+                                                                                                                 out_scale));
     return mixers_status();
 }
 

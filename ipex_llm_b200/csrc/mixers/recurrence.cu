@@ -7,6 +7,7 @@
 //   channel delta rule:      M <- diag(a) M;  u = beta (v - M^T k);  M <- M + k u^T;  o = M^T q   (a = exp(-exp(A) softplus(z + bias))
 //                                                                                                  per key channel)
 //   state-space scan:        M <- g M + dt k v^T;              o = M^T q + D v            (g = exp(-exp(A) dt), dt = softplus(. + bias))
+//   constant decay:          M <- g M + k v^T;                 o = M^T q                   (g a constant of the head; silu on q, k, v)
 // column j only needs k, q, the token's scalars and v_j.  So a column is owned by LPC lanes of a warp (LPC a power of two), each
 // holding R rows of it in registers for the whole call; tokens are taken in order.  Half of the block's warps own columns; the
 // other half stage the NEXT 16 tokens meanwhile in the second of two shared-memory buffers: their k / q (/ alpha) rows, scalars
@@ -88,6 +89,8 @@ struct RecArgs {
     const void* dt_bias;
     const void* z;          // gla, wkv, channel delta: decay logits [B, S, heads * dim]
     float inv_tau;
+    const float* decay;     // constant decay: one per head
+    int act_silu;           // constant decay: silu on q, k and v while they are staged
     const void* w0;         // wkv, channel delta: added to the decay logits [heads * dim]
     const void* u;          // wkv: the current token's bonus [heads * dim]; state-space scan: the skip weight D [heads]
     int B, S, heads, dim, vdim, slot0;
@@ -96,6 +99,9 @@ struct RecArgs {
     float* o;
     int lpc, tc;
 };
+
+// what q, k and v pass on their way into shared memory
+template <int MODE> __device__ __forceinline__ float rec_act(float z, int act_silu) { return MODE == 5 && act_silu ? silu_f(z) : z; }
 
 // shared memory of one stage: k, q (and alpha) rows of tc tokens padded to dp, the block's value columns, three scalars a token
 template <int MODE>
@@ -130,7 +136,7 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
         vreg[e] = 0.0f;
         if (i < nv) {
             int tt = i / cols_blk, cg = col0 + (i - tt * cols_blk);
-            if (cg < a.vdim) vreg[e] = to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * a.vdim + cg]);
+            if (cg < a.vdim) vreg[e] = rec_act<MODE>(to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * a.vdim + cg]), a.act_silu);
         }
     }
     float lb = 0.0f, la = 0.0f;                              // lane j: the gate logits of the warp's token j
@@ -161,7 +167,7 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
                 for (int e = 0; e < 4; ++e) {
                     const int i = blk + lane + 32 * e;
                     const bool ok = j < cnt && i < dim;
-                    qv[j][e] = ok ? to_f(row[a.off_q + qh * dim + i]) : 0.0f;
+                    qv[j][e] = ok ? to_f(row[a.off_q + qh * dim + i]) : 0.0f;         // constant decay: silu below, once all loads are out
                     kv[j][e] = ok ? to_f(row[a.off_k + qh * dim + i]) : 0.0f;
                     if (rec_decay_rows(MODE)) zv[j][e] = ok ? to_f(zr[i]) : 0.0f;
                 }
@@ -173,6 +179,7 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
                     for (int e = 0; e < 4; ++e) {
                         const int i = blk + lane + 32 * e;
                         if (i < dp) {
+                            if (MODE == 5) { qv[j][e] = rec_act<MODE>(qv[j][e], a.act_silu); kv[j][e] = rec_act<MODE>(kv[j][e], a.act_silu); }
                             if (MODE == 1) {
                                 st.a[(tt0 + j) * dp + i] = i < dim ? expf(log_sigmoid_f(zv[j][e]) * a.inv_tau) : 1.0f;
                                 st.q[(tt0 + j) * dp + i] = qv[j][e] * q_scale;
@@ -180,7 +187,7 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
                                 st.a[(tt0 + j) * dp + i] = i < dim ? expf(-expf(zv[j][e] + w0v[e])) : 1.0f;
                                 st.q[(tt0 + j) * dp + i] = qv[j][e];
                                 skq[j] += qv[j][e] * uv[e] * kv[j][e];
-                            } else if (MODE == 4) {
+                            } else if (MODE == 4 || MODE == 5) {
                                 st.q[(tt0 + j) * dp + i] = qv[j][e];
                             } else {
                                 if (MODE == 3) st.a[(tt0 + j) * dp + i] = i < dim ? expf(neg_exp_a * softplus_f(zv[j][e] + w0v[e])) : 1.0f;
@@ -231,7 +238,7 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
     }
     for (int i = ptid + VB * REC_PRODUCERS; i < nv; i += REC_PRODUCERS) {          // narrow heads only: more columns than one batch
         int tt = i / cols_blk, cg = col0 + (i - tt * cols_blk);
-        st.v[i] = cg < a.vdim ? to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * a.vdim + cg]) : 0.0f;
+        st.v[i] = cg < a.vdim ? rec_act<MODE>(to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * a.vdim + cg]), a.act_silu) : 0.0f;
     }
 }
 
@@ -240,7 +247,7 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
 // run 10 % slower); 2 halves them (some spills) so that two blocks hide each other's latencies, which pays when the grid has
 // more blocks than the GPU has SMs (batches, many heads): measured for the wkv mode only.
 template <typename T, int MODE, int R, int MINB>           // MODE 0: gated delta rule, 1: gated linear attention, 2: wkv,
-                                                           // 3: channel delta rule, 4: state-space scan
+                                                           // 3: channel delta rule, 4: state-space scan, 5: constant decay
 __global__ void __launch_bounds__(REC_THREADS, MINB) linear_recurrence_kernel(RecArgs a) {
     extern __shared__ float sh[];
     const int lpc = a.lpc, dp = R * lpc, tc = a.tc;
@@ -278,6 +285,7 @@ __global__ void __launch_bounds__(REC_THREADS, MINB) linear_recurrence_kernel(Re
         if (MODE != 3) dt_bias = to_f(((const T*)a.dt_bias)[h]);
     }
     const float skip = (MODE == 4 && !producer) ? to_f(((const T*)a.u)[h]) : 0.0f;
+    const float g_const = MODE == 5 ? a.decay[h] : 0.0f;
     if (producer && nchunks > 0)
         rec_stage_tokens<T, MODE>(a, RecStage<MODE>(sh, tc, dp, cols_blk), b, h, qh, first, (S - first < tc ? S - first : tc), dp, cols_blk, col0,
                                   tid - REC_CONSUMERS, neg_exp_a, dt_bias);
@@ -336,6 +344,12 @@ __global__ void __launch_bounds__(REC_THREADS, MINB) linear_recurrence_kernel(Re
                     o = (op[0] + op[1]) + (op[2] + op[3]);
                     for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
                     o += skip * v;
+                } else if (MODE == 5) {
+                    float op[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+                    for (int r = 0; r < R; ++r) { M[r] = g_const * M[r] + kr[r] * v; op[r & 3] += M[r] * qr[r]; }
+                    o = (op[0] + op[1]) + (op[2] + op[3]);
+                    for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
                 } else if (MODE == 1) {
                     const float* aa = st.a + tt * dp + sub;
                     float op[4] = {0.0f, 0.0f, 0.0f, 0.0f};
@@ -406,6 +420,7 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
         for (int t = 0; t < first; ++t) obase[(long)t * a.heads * vdim + col] = 0.0f;
     const float q_scale = rsqrtf((float)dim);
     const float skip = MODE == 4 ? to_f(((const T*)a.u)[h]) : 0.0f;
+    const float g_const = MODE == 5 ? a.decay[h] : 0.0f;
 
     for (int t0 = first; t0 < S; t0 += tc) {
         const int nt = S - t0 < tc ? S - t0 : tc;
@@ -417,7 +432,7 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
             const T* kr = row + a.off_k + qh * dim;
             float sq = 0.0f, sk = 0.0f, skq = 0.0f;
             for (int i = lane; i < dp; i += 32) {
-                float qv = i < dim ? to_f(qr[i]) : 0.0f, kv = i < dim ? to_f(kr[i]) : 0.0f;
+                const float qv = i < dim ? rec_act<MODE>(to_f(qr[i]), a.act_silu) : 0.0f, kv = i < dim ? rec_act<MODE>(to_f(kr[i]), a.act_silu) : 0.0f;
                 qbuf[tt * dp + i] = qv;
                 kbuf[tt * dp + i] = kv;
                 sq += qv * qv; sk += kv * kv; skq += qv * kv;
@@ -450,6 +465,8 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
                     sc[tt * 4 + 0] = expf(-expf(to_f(((const T*)a.A_log)[h])) * dt);
                     sc[tt * 4 + 1] = dt;
                 }
+            } else if (MODE == 5) {
+                // nothing but q, k and v
             } else if (MODE == 1) {
                 const T* zr = (const T*)a.z + ((long)b * S + t0 + tt) * ((long)a.heads * dim) + h * dim;
                 for (int i = lane; i < dp; i += 32) {
@@ -472,7 +489,7 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
         for (int i = tid; i < nt * cols_blk; i += REC_FEW_THREADS) {
             int tt = i / cols_blk, cl = i - tt * cols_blk;
             int cg = blockIdx.x * cols_blk + cl;
-            vbuf[i] = cg < vdim ? to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * vdim + cg]) : 0.0f;
+            vbuf[i] = cg < vdim ? rec_act<MODE>(to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * vdim + cg]), a.act_silu) : 0.0f;
         }
         __syncthreads();
         // ---- the tokens in order; a column's lanes only talk to each other
@@ -508,6 +525,11 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
                 for (int r = 0; r < R; ++r) { M[r] = g * M[r] + kk[r * lpc] * dv; o += M[r] * qq[r * lpc]; }
                 for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
                 o += skip * v;
+            } else if (MODE == 5) {
+                o = 0.0f;
+#pragma unroll
+                for (int r = 0; r < R; ++r) { M[r] = g_const * M[r] + kk[r * lpc] * v; o += M[r] * qq[r * lpc]; }
+                for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
             } else if (MODE == 1) {
                 const float* aa = abuf + tt * dp + sub;
                 o = 0.0f;
@@ -672,5 +694,18 @@ extern "C" int mixers_state_space_scan(int dtype, const void* conv, int B, int S
     a.proj = proj; a.ld_proj = ld; a.off_a = off_dt; a.A_log = A_log; a.dt_bias = dt_bias; a.u = skip;
     a.B = B; a.S = S; a.heads = heads; a.dim = n_state; a.vdim = vdim; a.slot0 = slot0; a.pad = pad; a.state = state; a.o = o;
     MIXERS_DISPATCH(dtype, return (launch_recurrence<T, 4>(a, (cudaStream_t)stream)));
+    return 0;
+}
+
+extern "C" int mixers_constant_decay_attention(int dtype, const void* proj, int B, int S, int ld, int off, int heads, int dim, int vdim,
+                                               const float* decay, int act_silu, float* state, int slot0, const int32_t* pad, float* o,
+                                               mixers_stream_t stream) {
+    if (B <= 0 || S <= 0) return 0;
+    if (!decay) return (int)cudaErrorInvalidValue;
+    RecArgs a = {};
+    a.src = proj; a.ld_src = ld; a.off_q = off; a.off_k = off + heads * dim; a.off_v = off + 2 * heads * dim; a.q_heads = heads;
+    a.decay = decay; a.act_silu = act_silu;
+    a.B = B; a.S = S; a.heads = heads; a.dim = dim; a.vdim = vdim; a.slot0 = slot0; a.pad = pad; a.state = state; a.o = o;
+    MIXERS_DISPATCH(dtype, return (launch_recurrence<T, 5>(a, (cudaStream_t)stream)));
     return 0;
 }

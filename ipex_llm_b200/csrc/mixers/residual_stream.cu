@@ -140,24 +140,32 @@ __global__ void rms_residual_cached_kernel(float* __restrict__ x, const TY* __re
 //   x += y_a + y_c + y_b + y_d (each may be null; y_a, y_c in the model's type, y_b, y_d 32-bit);
 //   pre_gain: x <- x / rms(x) * pre_gain[0] first (the norm behind an embedding);
 //   stack: the new x is kept as stream `index`, and with coef replaced by sum_{j <= index} coef[j] * stack[j];
-//   h1 = x / rms(x) * gain1[0], h2 = x / rms(x) * gain2[0] (either may be null): one root mean square serves both.
+//   h1 = x / rms(x) * gain1[0], h2 = x / rms(x) * gain2[0] (either may be null): one root mean square serves both;
+//   VEC: gain1 and gain2 are vectors [width] instead of one number each;
+//   replace: the stream is not added to but replaced by the sum of the addends (a stream that is projected anew);
+//   vec [width]: added to the sum (a vector that belongs to a pass over the layers);
+//   xc: the new x in the model's type, rows ld_xc apart (a column range of what the next projection reads).
 // CACHED: the row's elements stay in registers (rows up to SN_MAXC x blockDim wide), every load issued before the first reduction.
 constexpr int SN_MAXC = 8;
-template <typename T, bool CACHED>
+template <typename T, bool CACHED, bool VEC>
 __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, const T* __restrict__ y_a, const T* __restrict__ y_c,
                                           const float* __restrict__ y_b, const float* __restrict__ y_d, const T* __restrict__ pre_gain, float eps,
                                           float* __restrict__ stack, long stack_stride, int index, const T* __restrict__ coef,
-                                          const T* __restrict__ gain1, const T* __restrict__ gain2, T* __restrict__ h1, T* __restrict__ h2) {
+                                          const T* __restrict__ gain1, const T* __restrict__ gain2, T* __restrict__ h1, T* __restrict__ h2, int replace,
+                                          const T* __restrict__ vec, T* __restrict__ xc, long ld_xc) {
     __shared__ float red[32];
     const long base = (long)blockIdx.x * width;
+    const long base_c = (long)blockIdx.x * ld_xc;
     const bool want = h1 || h2;
     const float last = coef ? to_f(coef[index]) : 1.0f;
-    auto summed = [&](long i) {
-        float v = x[i];
+    auto summed = [&](int c) {
+        const long i = base + c;
+        float v = replace ? 0.0f : x[i];
         if (y_a) v += to_f(y_a[i]);
         if (y_c) v += to_f(y_c[i]);
         if (y_b) v += y_b[i];
         if (y_d) v += y_d[i];
+        if (vec) v += to_f(vec[c]);
         return v;
     };
     if (CACHED) {
@@ -166,9 +174,18 @@ __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, cons
 #pragma unroll
         for (int k = 0; k < SN_MAXC; ++k) {
             const int c = threadIdx.x + k * blockDim.x;
-            v[k] = c < width ? summed(base + c) : 0.0f;
+            v[k] = c < width ? summed(c) : 0.0f;
             av[k] = 0.0f;
             ss += v[k] * v[k];
+        }
+        float gv1[VEC ? SN_MAXC : 1], gv2[VEC ? SN_MAXC : 1];    // the norms' weights, on their way before the first reduction
+        if (VEC) {
+#pragma unroll
+            for (int k = 0; k < SN_MAXC; ++k) {
+                const int c = threadIdx.x + k * blockDim.x;
+                gv1[k % (VEC ? SN_MAXC : 1)] = h1 && c < width ? to_f(gain1[c]) : 0.0f;
+                gv2[k % (VEC ? SN_MAXC : 1)] = h2 && c < width ? to_f(gain2[c]) : 0.0f;
+            }
         }
         if (coef) {
             for (int j = 0; j < index; ++j) {
@@ -196,25 +213,26 @@ __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, cons
                     if (coef) v[k] = av[k] + last * v[k];
                 }
                 x[base + c] = v[k];
+                if (xc) xc[base_c + c] = from_f<T>(v[k]);
             }
             ss += v[k] * v[k];
         }
         if (!want) return;
         const float f = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
-        const float f1 = h1 ? f * to_f(gain1[0]) : 0.0f, f2 = h2 ? f * to_f(gain2[0]) : 0.0f;
+        const float f1 = VEC ? f : (h1 ? f * to_f(gain1[0]) : 0.0f), f2 = VEC ? f : (h2 ? f * to_f(gain2[0]) : 0.0f);
 #pragma unroll
         for (int k = 0; k < SN_MAXC; ++k) {
             const int c = threadIdx.x + k * blockDim.x;
             if (c < width) {
-                if (h1) h1[base + c] = from_f<T>(v[k] * f1);
-                if (h2) h2[base + c] = from_f<T>(v[k] * f2);
+                if (h1) h1[base + c] = from_f<T>(v[k] * f1 * (VEC ? gv1[k % (VEC ? SN_MAXC : 1)] : 1.0f));
+                if (h2) h2[base + c] = from_f<T>(v[k] * f2 * (VEC ? gv2[k % (VEC ? SN_MAXC : 1)] : 1.0f));
             }
         }
         return;
     }
     // every thread re-reads only what it wrote itself
     float ss = 0.0f;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) { const float v = summed(base + c); x[base + c] = v; ss += v * v; }
+    for (int c = threadIdx.x; c < width; c += blockDim.x) { const float v = summed(c); x[base + c] = v; ss += v * v; }
     const float f0 = pre_gain ? to_f(pre_gain[0]) / sqrtf(block_sum(ss, red) / (float)width + eps) : 1.0f;
     if (pre_gain || stack) {
         ss = 0.0f;
@@ -233,13 +251,15 @@ __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, cons
             ss += v * v;
         }
     }
+    if (xc)
+        for (int c = threadIdx.x; c < width; c += blockDim.x) xc[base_c + c] = from_f<T>(x[base + c]);
     if (!want) return;
     const float f = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
-    const float f1 = h1 ? f * to_f(gain1[0]) : 0.0f, f2 = h2 ? f * to_f(gain2[0]) : 0.0f;
+    const float f1 = VEC ? f : (h1 ? f * to_f(gain1[0]) : 0.0f), f2 = VEC ? f : (h2 ? f * to_f(gain2[0]) : 0.0f);
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         const float v = x[base + c];
-        if (h1) h1[base + c] = from_f<T>(v * f1);
-        if (h2) h2[base + c] = from_f<T>(v * f2);
+        if (h1) h1[base + c] = from_f<T>(v * f1 * (VEC ? to_f(gain1[c]) : 1.0f));
+        if (h2) h2[base + c] = from_f<T>(v * f2 * (VEC ? to_f(gain2[c]) : 1.0f));
     }
 }
 
@@ -399,19 +419,22 @@ extern "C" int mixers_clamped_glu(int dtype, const void* in, long n_rows, int ld
 
 extern "C" int mixers_sum_residual_norms(int dtype, float* x, long n_rows, int width, const void* y_a, const void* y_c, const float* y_b,
                                          const float* y_d, const void* pre_gain, float eps, float* stack, long stack_stride, int index,
-                                         const void* coef, const void* gain1, const void* gain2, void* h1, void* h2, mixers_stream_t stream) {
+                                         const void* coef, const void* gain1, const void* gain2, int gain_vectors, void* h1, void* h2, int replace,
+                                         const void* vec, void* xc, long ld_xc, mixers_stream_t stream) {
     if (n_rows <= 0) return 0;
-    if ((coef && !stack) || (h1 && !gain1) || (h2 && !gain2)) return (int)cudaErrorInvalidValue;
+    if ((xc && ld_xc < width) || (coef && !stack) || (h1 && !gain1) || (h2 && !gain2)) return (int)cudaErrorInvalidValue;
     int threads = width > 1024 ? 256 : 128;
     if (n_rows <= 64)                                        // a decoding step's few rows: one round trip to memory for rows up to 8192 wide
         while (threads < 1024 && threads * SN_MAXC < width) threads <<= 1;
     // many rows under a depth average stream better from the plain loop
     const bool cached = width <= SN_MAXC * threads && (n_rows <= 1024 || !coef);
-#define SN_LAUNCH(C) MIXERS_DISPATCH(dtype, sum_residual_norms_kernel<T, C><<<(unsigned)n_rows, threads, 0, (cudaStream_t)stream>>>(                    \
+#define SN_LAUNCH(C, V) MIXERS_DISPATCH(dtype, sum_residual_norms_kernel<T, C, V><<<(unsigned)n_rows, threads, 0, (cudaStream_t)stream>>>(              \
         x, width, (const T*)y_a, (const T*)y_c, y_b, y_d, (const T*)pre_gain, eps, stack, stack_stride, index, (const T*)coef, (const T*)gain1, \
-        (const T*)gain2, (T*)h1, (T*)h2))
-    if (cached) SN_LAUNCH(true);
-    else SN_LAUNCH(false);
+        (const T*)gain2, (T*)h1, (T*)h2, replace, (const T*)vec, (T*)xc, ld_xc))
+    if (cached && gain_vectors) SN_LAUNCH(true, true);
+    else if (cached) SN_LAUNCH(true, false);
+    else if (gain_vectors) SN_LAUNCH(false, true);
+    else SN_LAUNCH(false, false);
 #undef SN_LAUNCH
     return mixers_status();
 }

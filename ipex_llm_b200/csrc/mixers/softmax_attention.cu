@@ -141,11 +141,14 @@ __global__ void __launch_bounds__(QP_THREADS) wide_qkv_prepare_kernel(
 // rot_off + i + rot_dims / 2 (i < rot_dims / 2) and the pair (u, v) becomes (u cos a - v sin a, v cos a + u sin a) * amp with
 // a = position * inv_freq[i], the angle and its sine / cosine in double precision; the other channels pass unchanged.  The first
 // k_norm_cols channels of a key head are first divided by their root mean square and multiplied by k_norm_w (a latent that
-// shares its cache row with a rotated part).  Keys and values go to storage index held + t of caches given by three strides.
+// shares its cache row with a rotated part).  unit_rms: every query and key head is divided by its root mean square over the head
+// behind the rotation (no weight; a rotation keeps the sum of squares, so it is taken of what comes in, the rotated channels
+// counting amp^2 times).  Keys and values go to storage index held + t of caches given by three strides; off_v may equal off_k
+// (values that are the keys before norm and rotation).
 template <typename T>
 __global__ void rope_qk_prepare_kernel(const T* __restrict__ proj, int B, int S, int ld, int off_q, int off_k, int off_v, int heads, int kv_heads,
                                        int q_dim, int k_dim, int vdim, int q_rot_off, int k_rot_off, int rot_dims, const double* __restrict__ inv_freq,
-                                       float amp, const T* __restrict__ k_norm_w, int k_norm_cols, float eps, T* __restrict__ q_out,
+                                       float amp, const T* __restrict__ k_norm_w, int k_norm_cols, float eps, int unit_rms, T* __restrict__ q_out,
                                        T* __restrict__ k_store, long k_bs, long k_ps, long k_hs, T* __restrict__ v_store, long v_bs, long v_ps,
                                        long v_hs, int held, int shift, const int32_t* __restrict__ pad, const int32_t* __restrict__ dyn) {
     if (dyn) held = dyn[0];
@@ -177,6 +180,15 @@ __global__ void rope_qk_prepare_kernel(const T* __restrict__ proj, int B, int S,
         for (int c = lane; c < ncols; c += 32) { const float v = to_f(src[c]); ss += v * v; }
         inv = 1.0f / sqrtf(warp_sum(ss) / (float)ncols + eps);
     }
+    float unit = 1.0f;
+    if (unit_rms) {
+        float ss = 0.0f;
+        for (int c = lane; c < dim; c += 32) {
+            const float v = to_f(src[c]), w = (c >= rot_off && c < rot_off + rot_dims) ? amp : (c < ncols ? inv * to_f(k_norm_w[c]) : 1.0f);
+            ss += (v * w) * (v * w);
+        }
+        unit = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+    }
     const int half = rot_dims >> 1;
     const double dpos = (double)pos;
     for (int c = lane; c < dim; c += 32) {
@@ -193,7 +205,7 @@ __global__ void rope_qk_prepare_kernel(const T* __restrict__ proj, int B, int S,
             y = to_f(src[c]);
             if (c < ncols) y = y * inv * to_f(k_norm_w[c]);
         }
-        dst[c] = from_f<T>(pos >= 0 ? y : 0.0f);
+        dst[c] = from_f<T>(pos >= 0 ? y * unit : 0.0f);
     }
 }
 
@@ -872,7 +884,7 @@ extern "C" int mixers_wide_qkv_prepare(int dtype, const void* proj, int B, int S
 
 extern "C" int mixers_rope_qk_prepare(int dtype, const void* proj, int B, int S, int ld, int off_q, int off_k, int off_v, int heads, int kv_heads,
                                       int q_dim, int k_dim, int vdim, int q_rot_off, int k_rot_off, int rot_dims, const double* inv_freq, float amp,
-                                      const void* k_norm_w, int k_norm_cols, float eps, void* q_out, void* k_store, long k_bs, long k_ps,
+                                      const void* k_norm_w, int k_norm_cols, float eps, int unit_rms, void* q_out, void* k_store, long k_bs, long k_ps,
                                       long k_hs, void* v_store, long v_bs, long v_ps, long v_hs, int held, int shift, const int32_t* pad,
                                       const int32_t* dyn, mixers_stream_t stream) {
     if (B <= 0 || S <= 0) return 0;
@@ -883,7 +895,7 @@ extern "C" int mixers_rope_qk_prepare(int dtype, const void* proj, int B, int S,
     const unsigned blocks = (unsigned)((warps + 3) / 4);
     MIXERS_DISPATCH(dtype, rope_qk_prepare_kernel<T><<<blocks, 128, 0, (cudaStream_t)stream>>>(
         (const T*)proj, B, S, ld, off_q, off_k, off_v, heads, kv_heads, q_dim, k_dim, vdim, q_rot_off, k_rot_off, rot_dims, inv_freq, amp,
-        (const T*)k_norm_w, k_norm_cols, eps, (T*)q_out, (T*)k_store, k_bs, k_ps, k_hs, (T*)v_store, v_bs, v_ps, v_hs, held, shift, pad, dyn));
+        (const T*)k_norm_w, k_norm_cols, eps, unit_rms, (T*)q_out, (T*)k_store, k_bs, k_ps, k_hs, (T*)v_store, v_bs, v_ps, v_hs, held, shift, pad, dyn));
     return mixers_status();
 }
 

@@ -38,12 +38,13 @@ _SIGNATURES = {
                                                                    _c_ptr, _c_ptr],
     "mixers_state_space_scan": [_c_int, _c_ptr] + [_c_int] * 6 + [_c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr,
                                                                  _c_ptr, _c_ptr],
-    "mixers_sigmoid_gate": [_c_int, _c_ptr, _c_long, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr],
+    "mixers_sigmoid_gate": [_c_int, _c_ptr, _c_long, _c_long, _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_float, _c_ptr],
+    "mixers_constant_decay_attention": [_c_int, _c_ptr] + [_c_int] * 7 + [_c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_rms_pair_sum": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_float, _c_long, _c_int, _c_ptr, _c_ptr],
     "mixers_sum_residual_norms": [_c_int, _c_ptr, _c_long, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_long, _c_int,
-                                  _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr],
+                                  _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_long, _c_ptr],
     "mixers_gelu_erf": [_c_int, _c_ptr, _c_long, _c_ptr, _c_ptr],
-    "mixers_rope_qk_prepare": [_c_int, _c_ptr] + [_c_int] * 14 + [_c_ptr, _c_float, _c_ptr, _c_int, _c_float, _c_ptr, _c_ptr, _c_long, _c_long,
+    "mixers_rope_qk_prepare": [_c_int, _c_ptr] + [_c_int] * 14 + [_c_ptr, _c_float, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_long, _c_long,
                                                                  _c_long, _c_ptr, _c_long, _c_long, _c_long, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_moe_scatter_scaled": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_long, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "mixers_token_shift_mix": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr],

@@ -179,6 +179,11 @@ def _optimize_pre(model, qtype=None):
         # everything that reads a mixer's input (a parallel mixer: both branches' projections) -> one in_proj
         from ipex_llm_b200.transformers.models.nikedra import merge_projections
         model.apply(merge_projections)
+    elif model_type == "bugipel":
+        # everything that reads a mixer's input -> one in_proj; a parallel mixer's two output projections -> one out_proj
+        import functools
+        from ipex_llm_b200.transformers.models.bugipel import merge_projections
+        model.apply(functools.partial(merge_projections, row_multiple=128 if qtype is not None else 0))
     return model
 
 
@@ -210,7 +215,7 @@ def _optimize_post(model):
         convert_forward(model, module.MixtralRMSNorm, rms_norm_forward)
         convert_forward(model, module.MixtralModel, mixtral_model_forward)
         convert_forward(model, module.MixtralAttention, mixtral_attention_forward)
-    elif model_type in ("zafepel", "serotar", "zubedra", "nikedra"):
+    elif model_type in ("zafepel", "serotar", "zubedra", "nikedra", "bugipel"):
         # this package's own model class: its forwards already call the fused operators and pick the state cache;
         # the recorded decode step for such a cache goes behind generate()
         from ipex_llm_b200.transformers.state_decode_graph import install_state_generate

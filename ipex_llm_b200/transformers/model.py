@@ -39,7 +39,8 @@ def save_low_bit(self, save_dir, *args, **kwargs):
 NATIVE_ARCHITECTURES = {"Zafepel": "ipex_llm_b200.transformers.models.zafepel",
                         "Serotar": "ipex_llm_b200.transformers.models.serotar",
                         "Zubedra": "ipex_llm_b200.transformers.models.zubedra",
-                        "Nikedra": "ipex_llm_b200.transformers.models.nikedra"}
+                        "Nikedra": "ipex_llm_b200.transformers.models.nikedra",
+                        "Bugipel": "ipex_llm_b200.transformers.models.bugipel"}
 
 
 def native_architecture(model_dir):

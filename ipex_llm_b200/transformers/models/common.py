@@ -130,6 +130,18 @@ def merge_linear_inputs(linears: List[torch.nn.Linear]) -> torch.nn.Linear:
     return new_linear
 
 
+def zero_rows(like: torch.nn.Linear, rows_so_far: int, multiple: int):
+    """a bias-free projection of zeros that brings a merged row count up to a multiple (none when it is one already, or
+    when the multiple is 0): the low-bit prefill GEMM wants whole 128-row tiles"""
+    extra = -rows_so_far % multiple if multiple else 0
+    if not extra:
+        return []
+    with torch.device("meta"):
+        pad = torch.nn.Linear(1, 1, bias=False)
+    pad.weight = torch.nn.Parameter(torch.zeros(extra, like.weight.shape[1], dtype=like.weight.dtype, device=like.weight.device), requires_grad=False)
+    return [pad]
+
+
 def merge_qkv_base(module: torch.nn.Module, attention_class):
     """:40-53: q_proj, k_proj, v_proj -> qkv_proj on every attention module of the given class (or class name)"""
     if (isinstance(attention_class, str) and module.__class__.__name__ == attention_class

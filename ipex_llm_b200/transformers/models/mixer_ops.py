@@ -156,6 +156,19 @@ def gated_linear_attention(proj, heads, dim, vdim, z, tau, state, slot0, pad):
     return o
 
 
+def constant_decay_attention(proj, off, heads, dim, vdim, decay, state, slot0, pad, silu=True):
+    """linear attention with one constant decay per head over the new tokens (q | k | v in the columns of proj from ``off``, silu on
+    all three with ``silu``); decay fp32 [heads]; state fp32 [B, heads, dim, vdim] in place; returns o fp32 [B, S, heads, vdim]"""
+    B, S, P = proj.shape
+    invalidInputError(proj.is_contiguous() and off + heads * (2 * dim + vdim) <= P and decay.dtype == torch.float32 and decay.is_contiguous()
+                      and decay.numel() == heads and state.dtype == torch.float32 and state.is_contiguous()
+                      and state.shape == (B, heads, dim, vdim), "constant_decay_attention: unexpected layout")
+    o = torch.empty(B, S, heads, vdim, dtype=torch.float32, device=proj.device)
+    native.call("mixers_constant_decay_attention", native.dtype_code(proj.dtype), native.ptr(proj), B, S, P, int(off), heads, dim, vdim,
+                native.ptr(decay), int(bool(silu)), native.ptr(state), int(slot0), native.ptr(pad), native.ptr(o), native.stream(proj.device))
+    return o
+
+
 def gated_rms_norm(o, gate, off_g, weight, eps, out, out_col, out_scale, sigmoid=False, gate_first=False):
     """out[:, out_col:...] = out_scale * rms_norm(o per head) * weight * silu(gate columns from off_g); ``weight`` [vdim] serves
     every head, [heads * vdim] gives each head its own.  ``sigmoid``: the gate is sigmoid(.) instead of silu(.); ``gate_first``:
@@ -226,12 +239,13 @@ def wide_qkv_prepare(proj, off_q, off_k, off_v, heads, kv_heads, dim, vdim, q_w,
     return q
 
 
-def sigmoid_gate(o, gate, off_g, per_gate):
-    """o[n, c] *= sigmoid(gate[n, off_g + c // per_gate]) in place (o [N, C] contiguous, gate [N, P] contiguous)"""
-    invalidInputError(o.is_contiguous() and gate.is_contiguous() and o.dim() == 2 and gate.shape[0] == o.shape[0] and gate.dtype == o.dtype,
+def sigmoid_gate(o, gate, off_g, per_gate, scale=1.0):
+    """o[n, c] *= scale * sigmoid(gate[n, off_g + c // per_gate]) in place (o [N, C]: contiguous, or a column range of a contiguous
+    buffer; gate [N, P] contiguous)"""
+    invalidInputError(o.dim() == 2 and o.stride(1) == 1 and gate.is_contiguous() and gate.shape[0] == o.shape[0] and gate.dtype == o.dtype,
                       "sigmoid_gate: unexpected layout")
-    native.call("mixers_sigmoid_gate", native.dtype_code(o.dtype), native.ptr(o), o.shape[0], o.shape[1], native.ptr(gate), gate.shape[-1],
-                int(off_g), int(per_gate), native.stream(o.device))
+    native.call("mixers_sigmoid_gate", native.dtype_code(o.dtype), native.ptr(o), max(o.stride(0), o.shape[1]), o.shape[0], o.shape[1], native.ptr(gate),
+                gate.shape[-1], int(off_g), int(per_gate), float(scale), native.stream(o.device))
     return o
 
 
@@ -246,11 +260,14 @@ def rms_pair_sum(a, b, w_a, w_b, eps, scale):
     return out
 
 
-def sum_residual_norms(x, ys, out_dtype, eps, pre_gain=None, stack=None, index=0, coef=None, gain1=None, gain2=None):
+def sum_residual_norms(x, ys, out_dtype, eps, pre_gain=None, stack=None, index=0, coef=None, gain1=None, gain2=None, replace=False, vec=None,
+                       x_copy=None):
     """x += sum(ys) in place (x fp32 [N, W]; ``ys``: up to two tensors of the model's dtype and two fp32 ones); ``pre_gain``: x is
     first divided by its root mean square and multiplied by this scalar; with ``stack`` [streams, N, W] the new x is kept as
-    stream ``index`` and, with ``coef`` [index + 1], replaced by the coefficient-weighted sum of streams 0..index.  Returns
-    (x / rms(x) * gain1, x / rms(x) * gain2) in ``out_dtype`` (None where no gain is given)."""
+    stream ``index`` and, with ``coef`` [index + 1], replaced by the coefficient-weighted sum of streams 0..index.  ``replace``: the
+    sum of ``ys`` takes x's place; ``vec`` [W] is added with them; ``x_copy`` [N, W] (a column range of a wider buffer) receives the
+    new x in ``out_dtype``.  Gains are one number or a vector [W].  Returns (x / rms(x) * gain1, x / rms(x) * gain2) in
+    ``out_dtype`` (None where no gain is given)."""
     n, w = x.shape
     invalidInputError(x.dtype == torch.float32 and x.is_contiguous(), "sum_residual_norms: x is a contiguous fp32 [N, W]")
     ys = [y for y in ys if y is not None]
@@ -264,12 +281,19 @@ def sum_residual_norms(x, ys, out_dtype, eps, pre_gain=None, stack=None, index=0
     invalidInputError(stack is None or (stack.dtype == torch.float32 and stack.is_contiguous() and stack.shape[1:] == x.shape and index < stack.shape[0]),
                       "sum_residual_norms: the kept streams are a contiguous fp32 [streams, N, W]")
     invalidInputError(coef is None or (stack is not None and coef.numel() == index + 1), "sum_residual_norms: one coefficient per kept stream")
+    gains = [t for t in (gain1, gain2) if t is not None]
+    vectors = bool(gains) and gains[0].numel() == w and gains[0].dim() == 1
+    invalidInputError(all(t.dtype == out_dtype and t.is_contiguous() and t.numel() == (w if vectors else 1) for t in gains)
+                      and (vec is None or (vec.dtype == out_dtype and vec.numel() == w and vec.is_contiguous()))
+                      and (x_copy is None or (x_copy.shape == x.shape and x_copy.dtype == out_dtype and x_copy.stride(1) == 1)),
+                      "sum_residual_norms: gains are one number each or vectors [W]; the vector and the copy have the model's dtype")
     typed, floats = typed + [None, None], floats + [None, None]
     h1 = torch.empty(n, w, dtype=out_dtype, device=x.device) if gain1 is not None else None
     h2 = torch.empty(n, w, dtype=out_dtype, device=x.device) if gain2 is not None else None
     native.call("mixers_sum_residual_norms", native.dtype_code(out_dtype), native.ptr(x), n, w, native.ptr(typed[0]), native.ptr(typed[1]),
                 native.ptr(floats[0]), native.ptr(floats[1]), native.ptr(pre_gain), float(eps), native.ptr(stack), n * w, int(index),
-                native.ptr(coef), native.ptr(gain1), native.ptr(gain2), native.ptr(h1), native.ptr(h2), native.stream(x.device))
+                native.ptr(coef), native.ptr(gain1), native.ptr(gain2), int(vectors), native.ptr(h1), native.ptr(h2), int(bool(replace)), native.ptr(vec),
+                native.ptr(x_copy), max(x_copy.stride(0), w) if x_copy is not None else w, native.stream(x.device))
     return h1, h2
 
 
@@ -282,11 +306,12 @@ def gelu_erf(z):
 
 
 def rope_qk_prepare(proj, off_q, off_k, off_v, heads, kv_heads, q_dim, k_dim, vdim, q_rot_off, k_rot_off, rot_dims, inv_freq, amp, k_store,
-                    k_strides, v_store, v_strides, held, shift, pad, eps=0.0, k_norm_w=None, k_norm_cols=0, dyn=None):
+                    k_strides, v_store, v_strides, held, shift, pad, eps=0.0, k_norm_w=None, k_norm_cols=0, dyn=None, unit_rms=False):
     """rotary positions on the new tokens' queries and keys (columns of proj [B, S, P]) and the cache write of keys and values;
     ``k_strides`` / ``v_strides``: (batch, position, head) strides of the caches in elements; ``inv_freq`` float64 [rot_dims / 2],
     ``amp`` multiplies cosine and sine; ``k_norm_w``: the first ``k_norm_cols`` channels of every key head are RMS-normalised with
-    this weight.  Returns q [B * S, heads * q_dim]"""
+    this weight; ``unit_rms``: behind the rotation every query and key head is divided by its root mean square.  Returns q
+    [B * S, heads * q_dim]"""
     B, S, P = proj.shape
     invalidInputError(proj.is_contiguous() and k_store.dtype == proj.dtype and (v_store is None or v_store.dtype == proj.dtype)
                       and (rot_dims == 0 or (inv_freq.dtype == torch.float64 and inv_freq.numel() == rot_dims // 2 and inv_freq.is_contiguous())),
@@ -295,7 +320,7 @@ def rope_qk_prepare(proj, off_q, off_k, off_v, heads, kv_heads, q_dim, k_dim, vd
     vs = v_strides if v_store is not None else (0, 0, 0)
     native.call("mixers_rope_qk_prepare", native.dtype_code(proj.dtype), native.ptr(proj), B, S, P, int(off_q), int(off_k), int(off_v), heads, kv_heads,
                 q_dim, k_dim, vdim if v_store is not None else 0, int(q_rot_off), int(k_rot_off), int(rot_dims), native.ptr(inv_freq) if rot_dims else None,
-                float(amp), native.ptr(k_norm_w), int(k_norm_cols), float(eps), native.ptr(q), native.ptr(k_store), *[int(v) for v in k_strides],
+                float(amp), native.ptr(k_norm_w), int(k_norm_cols), float(eps), int(bool(unit_rms)), native.ptr(q), native.ptr(k_store), *[int(v) for v in k_strides],
                 native.ptr(v_store), *[int(v) for v in vs], int(held), int(shift), native.ptr(pad), native.ptr(dyn), native.stream(proj.device))
     return q
 

@@ -25,7 +25,6 @@ them like any other model's.  The residual stream and the kept streams, every no
 and weights and everything inside the recurrences are 32-bit whatever the model's dtype.
 """
 import json
-import math
 import os
 from typing import Optional
 
@@ -37,12 +36,13 @@ from transformers.modeling_outputs import CausalLMOutputWithPast
 from ipex_llm_b200.transformers.kv import DynamicStateCache
 from ipex_llm_b200.transformers.models import experts, mixer_ops as ops
 from ipex_llm_b200.transformers.models.common import merge_linear
+from ipex_llm_b200.transformers.models.mixers import (ChannelDeltaMixer, Rotary, Weight, channel_delta, plain_linears, rotary_frequencies,  # noqa: F401
+                                                      short_conv)
 from ipex_llm_b200.transformers.models.utils import read_safetensors
 from ipex_llm_b200.utils.common import invalidInputError
 
 ABSORB_MAX_TOKENS = 16        # up to this many new tokens per row attend to the latent cache itself (no key / value expansion)
 OVERLAP_MIN_TOKENS = 256      # from this many new tokens on, a layer's feed-forward runs on a second stream beside its mixer
-YARN_AMP_SLOPE = 0.1          # cosine and sine of rescaled frequencies are multiplied by slope * ln(factor) + 1
 
 
 class NikedraConfig(PreTrainedConfig):
@@ -75,74 +75,6 @@ class NikedraConfig(PreTrainedConfig):
         return int(self.canon["taps"])
 
 
-def rotary_frequencies(rot):
-    """(frequency of every rotated pair as a list of floats, amplitude) of a ``rot`` block: base^(-2i / dims); with ``scaling``
-    (factor, original, fast, slow) a pair whose wavelength makes fewer than ``slow`` turns within ``original`` positions is slowed
-    down by ``factor``, one that makes more than ``fast`` turns is kept, the pairs between are blended linearly by their index,
-    and cosine and sine are multiplied by 0.1 ln(factor) + 1"""
-    dims, base = int(rot["dims"]), float(rot["base"])
-    freq = [base ** (-2.0 * i / dims) for i in range(dims // 2)]
-    sc = rot.get("scaling")
-    if not sc:
-        return freq, 1.0
-    factor, original = float(sc["factor"]), float(sc["original"])
-
-    def pair_with_turns(turns):                              # the (fractional) pair index whose wavelength makes this many turns
-        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
-
-    lo = max(math.floor(pair_with_turns(float(sc["fast"]))), 0)
-    hi = min(math.ceil(pair_with_turns(float(sc["slow"]))), dims - 1)
-    out = []
-    for i, f in enumerate(freq):
-        ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
-        out.append(f / factor * ramp + f * (1.0 - ramp))
-    return out, YARN_AMP_SLOPE * math.log(factor) + 1.0
-
-
-class _Rotary:
-    """frequencies of a ``rot`` block in double precision on the device they are needed on (not a buffer: ``model.to(dtype)`` must
-    not round them; the kernel forms the angles in double precision too)"""
-
-    def __init__(self, rot):
-        self.dims = int(rot["dims"])
-        invalidInputError(self.dims % 2 == 0, "rotary dims must be even")
-        self.freq, self.amp = rotary_frequencies(rot)
-        self._on = {}
-
-    def inv_freq(self, device):
-        t = self._on.get(device)
-        if t is None:
-            t = self._on[device] = torch.tensor(self.freq or [0.0], dtype=torch.float64).to(device)
-        return t
-
-
-class _Weight(nn.Module):
-    """a lone parameter under the name ``<module>.weight``: a norm's vector of weights, or (shape ()) its single gain"""
-
-    def __init__(self, *shape):
-        super().__init__()
-        self.weight = nn.Parameter(torch.ones(tuple(shape)))
-
-
-class ChannelDeltaMixer(nn.Module):
-    """``q_proj`` .. ``g1_proj`` (everything that reads the mixer's input) become one ``in_proj`` when ``merge_projections`` has run"""
-    PARTS = ("q_proj", "k_proj", "v_proj", "b_proj", "a1_proj", "g1_proj")
-
-    def __init__(self, width, m, ranks):
-        super().__init__()
-        self.heads, self.kv_heads, self.dim, self.vdim, self.taps = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"])
-        invalidInputError(self.kv_heads >= 1 and self.heads % self.kv_heads == 0, "heads must be a multiple of kv_heads")
-        qk, v = self.kv_heads * self.dim, self.heads * self.vdim
-        self.q_proj, self.k_proj, self.v_proj = nn.Linear(width, qk, bias=False), nn.Linear(width, qk, bias=False), nn.Linear(width, v, bias=False)
-        self.b_proj = nn.Linear(width, self.heads, bias=False)
-        self.a1_proj, self.a2_proj = nn.Linear(width, ranks[0], bias=False), nn.Linear(ranks[0], self.heads * self.dim, bias=False)
-        self.g1_proj, self.g2_proj = nn.Linear(width, ranks[1], bias=False), nn.Linear(ranks[1], v, bias=False)
-        self.conv_weight = nn.Parameter(torch.zeros(2 * qk + v, self.taps))          # q | k | v channels
-        self.A_log, self.dt_bias = nn.Parameter(torch.zeros(self.heads)), nn.Parameter(torch.zeros(self.heads * self.dim))
-        self.norm = _Weight(self.vdim)
-        self.o_proj = nn.Linear(v, width, bias=False)
-
-
 class LatentRopeAttention(nn.Module):
     """``q_proj`` / ``dkv`` / ``g_proj`` become one ``in_proj`` when ``merge_projections`` has run.  A cache row is [latent | rotated
     key part]; ``expand`` [heads * (dim + rot_dim) + heads * vdim, kv_rank + rot_dim] turns such rows into every head's key
@@ -154,13 +86,13 @@ class LatentRopeAttention(nn.Module):
         super().__init__()
         self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = (int(m[k]) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
         self.scale, self.window = float(m["scale"]), int(m["mask"]["size"])
-        self.rotary = _Rotary(dict(m["rot"], dims=self.rot_dim))
+        self.rotary = Rotary(dict(m["rot"], dims=self.rot_dim))
         qd = self.dim + self.rot_dim
         self.q_proj = nn.Linear(width, self.heads * qd, bias=False)
         self.dkv = nn.Linear(width, self.kv_rank + self.rot_dim, bias=False)
         self.g_proj = nn.Linear(width, self.heads * self.vdim, bias=False)
-        self.dkv_norm = _Weight(self.kv_rank)
-        self.expand = _Weight(self.heads * (qd + self.vdim), self.kv_rank + self.rot_dim)
+        self.dkv_norm = Weight(self.kv_rank)
+        self.expand = Weight(self.heads * (qd + self.vdim), self.kv_rank + self.rot_dim)
         self.o_proj = nn.Linear(self.heads * self.vdim, width, bias=False)
 
     def expansion(self, uk, uv):
@@ -180,14 +112,14 @@ class ChunkedAttention(nn.Module):
         self.heads, self.kv_heads, self.dim, self.vdim = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
         invalidInputError(self.kv_heads >= 1 and self.heads % self.kv_heads == 0, "heads must be a multiple of kv_heads")
         self.scale, self.chunk = float(m["scale"]), int(m["mask"]["size"])
-        self.rotary = _Rotary(m["rot"])
+        self.rotary = Rotary(m["rot"])
         invalidInputError(self.rotary.dims <= self.dim, "rotary dims exceed the head size")
         self.q_proj = nn.Linear(width, self.heads * self.dim, bias=False)
         self.k_proj = nn.Linear(width, self.kv_heads * self.dim, bias=False)
         self.v_proj = nn.Linear(width, self.kv_heads * self.vdim, bias=False)
         self.g_proj = nn.Linear(width, self.heads, bias=False)
         self.o_proj = nn.Linear(self.heads * self.vdim, width, bias=False)
-        self.out = _Weight(width)
+        self.out = Weight(width)
 
 
 class StateSpaceMixer(nn.Module):
@@ -204,9 +136,9 @@ class StateSpaceMixer(nn.Module):
         self.in_proj = nn.Linear(width, 2 * self.inner + 2 * self.groups * self.state + self.heads, bias=False)
         self.conv_weight, self.conv_bias = nn.Parameter(torch.zeros(self.conv_channels, self.taps)), nn.Parameter(torch.zeros(self.conv_channels))
         self.dt_bias, self.A_log, self.D = (nn.Parameter(torch.zeros(self.heads)) for _ in range(3))
-        self.norm = _Weight(self.inner)
+        self.norm = Weight(self.inner)
         self.o_proj = nn.Linear(self.inner, width, bias=False)
-        self.out = _Weight(width)
+        self.out = Weight(width)
 
 
 class ParallelMixer(nn.Module):
@@ -261,7 +193,7 @@ class NikedraLayer(nn.Module):
         lc, w = config.layers[index], config.width
         self.kind = lc["type"]
         invalidInputError(self.kind in MIXER_TYPES, f"unknown layer type {self.kind}")
-        self.norm1 = _Weight()
+        self.norm1 = Weight()
         self.canon = nn.Parameter(torch.zeros(w, config.canon_taps))
         if self.kind == "channel_delta":
             self.mixer = ChannelDeltaMixer(w, lc["mixer"], config.low_ranks.get(str(index), [1, 1]))
@@ -275,7 +207,7 @@ class NikedraLayer(nn.Module):
             kind = m.get("kind", "dense")
             invalidInputError(kind in ("dense", "moe"), f"unknown feed-forward kind {kind}")
             self.mlp = ClampedMLP(w, m) if kind == "dense" else InputWeightedExperts(w, m)
-            self.norm2 = _Weight()
+            self.norm2 = Weight()
         self.dwa = nn.Parameter(torch.ones(index + 2))
 
 
@@ -299,9 +231,9 @@ class NikedraModel(nn.Module):
         super().__init__()
         self.config = config
         self.embed_tokens = nn.Embedding(config.vocab, config.width)
-        self.embed_norm = _Weight()
+        self.embed_norm = Weight()
         self.layers = nn.ModuleList([NikedraLayer(config, i) for i in range(len(config.layers))])
-        self.norm = _Weight()
+        self.norm = Weight()
 
 
 class NikedraForCausalLM(PreTrainedModel, GenerationMixin):
@@ -329,45 +261,11 @@ class NikedraForCausalLM(PreTrainedModel, GenerationMixin):
     def get_output_embeddings(self):
         return self.lm_head
 
-    # ---- helpers
-    def _plain_linears(self):
-        """no projection was converted to a low-bit format (those products share one workspace per device, so two of them
-        must not run on two streams at once)"""
-        plain = self.__dict__.get("_b200_plain_linears")
-        if plain is None:
-            plain = self.__dict__["_b200_plain_linears"] = all(type(m) is nn.Linear for m in self.modules() if isinstance(m, nn.Linear) or
-                                                               type(m).__name__ == "LowBitLinear")
-        return plain
-
-    @staticmethod
-    def _conv(proj, off, channels, weight, bias, rec, key, B, S, cache, silu, add_input=False):
-        """a short causal convolution over the new tokens and the state's tail (which keeps its address: a recorded step holds it)"""
-        taps = weight.shape[1]
-        tail, tail_next = rec.tails(B, taps, channels, proj.dtype, proj.device, key=key)
-        pad = cache.pad if cache.seen == 0 else None                         # padding only ever precedes a row's first call
-        y = ops.short_conv(proj, off, channels, weight, bias, tail, tail if S == 1 else tail_next, cache.seen, pad, silu=silu, add_input=add_input)
-        if S > 1:
-            tail.copy_(tail_next)
-        return y
-
     # ---- mixers (h: the mixer's input in the model's dtype, [N, W]); each returns [N, W]
     def _channel_delta(self, mx, h, st, B, S, cache):
         invalidInputError(hasattr(mx, "in_proj"), "the mixers' projections are merged at load time (merge_projections)")
-        H, G, D, Dv = mx.heads, mx.kv_heads, mx.dim, mx.vdim
-        proj = mx.in_proj(h)                                                 # q | k | v | beta | decay rank | gate rank
-        P = proj.shape[1]
-        C = 2 * G * D + H * Dv
-        off_b = C
-        off_a1 = off_b + H
-        off_g1 = off_a1 + mx.a2_proj.in_features
-        conv = self._conv(proj.view(B, S, P), 0, C, mx.conv_weight, None, st.rec, "mixer", B, S, cache, silu=True)
-        z = mx.a2_proj(proj[:, off_a1:off_g1])                               # decay logits [N, H D]
-        gate = mx.g2_proj(proj[:, off_g1:off_g1 + mx.g2_proj.in_features])   # [N, H Dv]
-        state = st.rec.matrix(B, H, D, Dv, h.device)
-        o = ops.channel_delta_rule(conv, G, H, D, Dv, proj.view(B, S, P), off_b, z, mx.A_log, mx.dt_bias, state, cache.seen,
-                                   cache.pad if cache.seen == 0 else None)
-        out = torch.empty(B * S, H * Dv, dtype=h.dtype, device=h.device)
-        ops.gated_rms_norm(o, gate, 0, mx.norm.weight, self.config.norm_eps, out, 0, 1.0, sigmoid=True)
+        out = torch.empty(B * S, mx.heads * mx.vdim, dtype=h.dtype, device=h.device)
+        channel_delta(mx, mx.in_proj(h), 0, st.rec, B, S, cache, self.config.norm_eps, out)
         return mx.o_proj(out)
 
     def _latent_attention(self, mx, h, st, B, S, cache):
@@ -440,7 +338,7 @@ class NikedraForCausalLM(PreTrainedModel, GenerationMixin):
         ops.sigmoid_gate(o, proj, off_g, Dv)
         left = l.o_proj(o)
         # right: convolution over x | B | C, the scan, the gate, the grouped norm
-        conv = self._conv(proj3, off_x, r.conv_channels, r.conv_weight, r.conv_bias, st.rec, "mixer", B, S, cache, silu=True)
+        conv = short_conv(proj3, off_x, r.conv_channels, r.conv_weight, r.conv_bias, st.rec, "mixer", B, S, cache, silu=True)
         state = st.rec.matrix(B, r.heads, r.state, r.vdim, h.device)
         y = ops.state_space_scan(conv, r.groups, r.heads, r.state, r.vdim, proj3, off_dt, r.A_log, r.dt_bias, r.D, state, cache.seen,
                                  cache.pad if cache.seen == 0 else None)
@@ -496,7 +394,7 @@ class NikedraForCausalLM(PreTrainedModel, GenerationMixin):
 
         main = side = forked = None
         if (self.overlap_feed_forward and B * S >= OVERLAP_MIN_TOKENS and dev.type == "cuda" and not cache.frozen
-                and not torch.cuda.is_current_stream_capturing() and self._plain_linears()):
+                and not torch.cuda.is_current_stream_capturing() and plain_linears(self)):
             main = torch.cuda.current_stream(dev)
             if self._side_stream is None or self._side_stream.device != dev:
                 self._side_stream = torch.cuda.Stream(dev)
@@ -510,7 +408,7 @@ class NikedraForCausalLM(PreTrainedModel, GenerationMixin):
                 st = cache.run_state(i, window=0 if layer.kind == "parallel" else None)
             if side is not None and layer.mlp is not None:
                 forked = main.record_event()                                 # h2 is ready here; nothing of this layer's mixer is queued yet
-            hm = self._conv(h1.view(B, S, -1), 0, cfg.width, layer.canon, None, st.rec, "input", B, S, cache, silu=False, add_input=True)
+            hm = short_conv(h1.view(B, S, -1), 0, cfg.width, layer.canon, None, st.rec, "input", B, S, cache, silu=False, add_input=True)
             hm = hm.view(B * S, -1)
             if layer.kind == "channel_delta":
                 y_mix = self._channel_delta(layer.mixer, hm, st, B, S, cache)

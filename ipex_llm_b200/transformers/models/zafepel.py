@@ -24,7 +24,7 @@ from transformers.modeling_outputs import CausalLMOutputWithPast
 
 from ipex_llm_b200.transformers.kv import DynamicStateCache
 from ipex_llm_b200.transformers.models import mixer_ops as ops
-from ipex_llm_b200.transformers.models.common import merge_linear, merge_linear_inputs
+from ipex_llm_b200.transformers.models.common import merge_linear, merge_linear_inputs, zero_rows
 from ipex_llm_b200.transformers.models.utils import read_safetensors
 from ipex_llm_b200.utils.common import invalidInputError
 
@@ -176,17 +176,6 @@ class ZafepelLayer(nn.Module):
             self.mlp = PolyNormMLP(width, lc["mlp"])
 
 
-def _zero_rows(like: nn.Linear, rows_so_far: int, multiple: int):
-    """a bias-free projection of zeros that brings a merged row count up to a multiple (none when it is one already)"""
-    extra = -rows_so_far % multiple if multiple else 0
-    if not extra:
-        return []
-    with torch.device("meta"):
-        pad = nn.Linear(1, 1, bias=False)
-    pad.weight = nn.Parameter(torch.zeros(extra, like.weight.shape[1], dtype=like.weight.dtype, device=like.weight.device), requires_grad=False)
-    return [pad]
-
-
 def merge_projections(module: nn.Module, row_multiple: int = 0):
     """every projection that reads the mixer's input becomes one ``in_proj``; the two output projections of a parallel mixer
     become one ``out_proj`` over the concatenated branch outputs.  ``row_multiple``: rows of zeros are appended to ``in_proj`` up
@@ -195,12 +184,12 @@ def merge_projections(module: nn.Module, row_multiple: int = 0):
     if isinstance(module, ParallelMixer) and not hasattr(module, "in_proj"):
         l, r = module.left, module.right
         parts = [l.q_proj, l.k_proj, l.v_proj, r.q_proj, r.k_proj, r.v_proj, r.b_proj, r.a_proj, r.g_proj]
-        module.in_proj = merge_linear(parts + _zero_rows(l.q_proj, sum(p.weight.shape[0] for p in parts), row_multiple))
+        module.in_proj = merge_linear(parts + zero_rows(l.q_proj, sum(p.weight.shape[0] for p in parts), row_multiple))
         module.out_proj = merge_linear_inputs([l.o_proj, r.o_proj])
         del l.q_proj, l.k_proj, l.v_proj, l.o_proj, r.q_proj, r.k_proj, r.v_proj, r.b_proj, r.a_proj, r.g_proj, r.o_proj
     elif isinstance(module, GatedLinearAttention) and not hasattr(module, "in_proj"):
         parts = [module.q_proj, module.k_proj, module.v_proj, module.g_proj, module.a1_proj]
-        module.in_proj = merge_linear(parts + _zero_rows(module.q_proj, sum(p.weight.shape[0] for p in parts), row_multiple))
+        module.in_proj = merge_linear(parts + zero_rows(module.q_proj, sum(p.weight.shape[0] for p in parts), row_multiple))
         del module.q_proj, module.k_proj, module.v_proj, module.g_proj, module.a1_proj
 
 
