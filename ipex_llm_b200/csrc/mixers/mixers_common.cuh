@@ -28,6 +28,27 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : lo
 // log(sigmoid(z)) without cancellation on either side
 __device__ __forceinline__ float log_sigmoid_f(float z) { return z >= 0.0f ? -log1pf(expf(-z)) : z - log1pf(expf(z)); }
 
+// four neighbours at once (the address a multiple of four elements)
+template <typename T> __device__ __forceinline__ float4 load4(const T* p) {
+    if constexpr (sizeof(T) == 4) {
+        return *reinterpret_cast<const float4*>(p);
+    } else {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        const T* e = reinterpret_cast<const T*>(&u);
+        return make_float4(to_f(e[0]), to_f(e[1]), to_f(e[2]), to_f(e[3]));
+    }
+}
+template <typename T> __device__ __forceinline__ void store4(T* p, float4 v) {
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(p) = v;
+    } else {
+        uint2 u;
+        T* e = reinterpret_cast<T*>(&u);
+        e[0] = from_f<T>(v.x); e[1] = from_f<T>(v.y); e[2] = from_f<T>(v.z); e[3] = from_f<T>(v.w);
+        *reinterpret_cast<uint2*>(p) = u;
+    }
+}
+
 // q (32-bit, e.g. staged in shared memory) . one row of keys; 16-byte loads when the rows allow them
 template <typename T>
 __device__ __forceinline__ float dot_row(const float* __restrict__ qs, const T* __restrict__ kr, int dim) {

@@ -177,6 +177,45 @@ __global__ void gated_rms_norm_wide_kernel(const float* __restrict__ o, int head
     }
 }
 
+// the same for heads that come in groups of four channels: a thread owns up to K groups and moves each as one word
+template <typename T, int K>
+__global__ void gated_rms_norm_wide4_kernel(const float* __restrict__ o, int heads, int vdim, const T* __restrict__ gate, int ld_gate, int off_g,
+                                            const T* __restrict__ w, int w_head_stride, float eps, T* __restrict__ out, int ld_out, int out_col,
+                                            float out_scale, int gate_mode) {
+    __shared__ float red[32];
+    const long item = blockIdx.x;
+    const long n = item / heads;
+    const int h = (int)(item - n * heads);
+    const float* src = o + item * (long)vdim;
+    const T* g = gate + n * (long)ld_gate + off_g + h * vdim;
+    w += (long)h * w_head_stride;
+    const bool first = (gate_mode & 2) != 0;
+    auto act = [&](float z) { return (gate_mode & 1) ? sigmoid_f(z) : silu_f(z); };
+    float4 v[K], gt[K], wt[K];
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+        const int c = 4 * (threadIdx.x + k * blockDim.x);
+        v[k] = gt[k] = wt[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (c < vdim) { v[k] = load4(src + c); gt[k] = load4(g + c); wt[k] = load4(w + c); }
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+        gt[k] = make_float4(act(gt[k].x), act(gt[k].y), act(gt[k].z), act(gt[k].w));
+        const float4 t = make_float4(v[k].x * gt[k].x, v[k].y * gt[k].y, v[k].z * gt[k].z, v[k].w * gt[k].w);
+        const float4 u = first ? t : v[k];
+        ss += (u.x * u.x + u.y * u.y) + (u.z * u.z + u.w * u.w);
+        v[k] = t;
+    }
+    const float inv = out_scale / sqrtf(gn_block_sum(ss, red) / (float)vdim + eps);
+    T* dst = out + n * (long)ld_out + out_col + h * vdim;
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+        const int c = 4 * (threadIdx.x + k * blockDim.x);
+        if (c < vdim) store4(dst + c, make_float4(v[k].x * inv * wt[k].x, v[k].y * inv * wt[k].y, v[k].z * inv * wt[k].z, v[k].w * inv * wt[k].w));
+    }
+}
+
 // o[n, c] *= out_scale * sigmoid(gate[n, off_g + c / per_gate]) in place (o: rows of `cols` channels, ld_o apart): a gate per channel
 // (per_gate 1) or one per head (per_gate = the head's channels)
 template <typename T>
@@ -291,11 +330,23 @@ extern "C" int mixers_gated_rms_norm(int dtype, const float* o, long n_rows, int
     if (n_rows <= 0) return 0;
     if (gate_mode & ~3) return (int)cudaErrorInvalidValue;
     long warps = n_rows * heads;
-    if (vdim > 256 && vdim <= GN_MAXC * 1024 && warps <= 1024) {   // few wide heads (a decoding step): a block each; many rows keep every SM
-                                                                    // busy with a warp each
+    const uintptr_t halves = (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out;
+    if (vdim > 256 && vdim <= 8192 && (warps <= 1024 || vdim >= 512) && ((vdim | ld_gate | off_g | w_head_stride | ld_out | out_col) & 3) == 0 &&
+        ((uintptr_t)o & 15) == 0 && (halves & (dtype == 0 ? 15 : 7)) == 0) {
+        const int groups = vdim / 4, one = (groups + 31) / 32 * 32, two = ((groups + 1) / 2 + 31) / 32 * 32;
+#define GN4_LAUNCH(K, TH) MIXERS_DISPATCH(dtype, gated_rms_norm_wide4_kernel<T, K><<<(unsigned)warps, TH, 0, (cudaStream_t)stream>>>( \
+        o, heads, vdim, (const T*)gate, ld_gate, off_g, (const T*)w, w_head_stride, eps, (T*)out, ld_out, out_col, out_scale, gate_mode))
+        if (one <= 1024 && (warps <= 64 || one <= 128)) GN4_LAUNCH(1, one);
+        else GN4_LAUNCH(2, two);
+#undef GN4_LAUNCH
+        return mixers_status();
+    }
+    // a block per wide head: always from 1024 channels on (a warp would walk 32 and more values a lane twice), for narrower ones when
+    // there are few of them (a decoding step); many narrow heads keep every SM busy with a warp each
+    if (vdim > 256 && vdim <= GN_MAXC * 1024 && (warps <= 1024 || vdim >= 1024)) {
         int threads = 128;
         while (threads < 1024 && threads * GN_MAXC < vdim) threads <<= 1;
-        if (threads * 4 <= vdim && threads < 1024) threads <<= 1;   // at least two rounds of loads in flight per thread are enough
+        if (warps <= 1024 && threads * 4 <= vdim && threads < 1024) threads <<= 1;   // at least two rounds of loads in flight per thread are enough
         MIXERS_DISPATCH(dtype, gated_rms_norm_wide_kernel<T><<<(unsigned)warps, threads, 0, (cudaStream_t)stream>>>(
             o, heads, vdim, (const T*)gate, ld_gate, off_g, (const T*)w, w_head_stride, eps, (T*)out, ld_out, out_col, out_scale, gate_mode));
         return mixers_status();

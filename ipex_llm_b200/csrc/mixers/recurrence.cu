@@ -9,8 +9,8 @@
 //   state-space scan:        M <- g M + dt k v^T;              o = M^T q + D v            (g = exp(-exp(A) dt), dt = softplus(. + bias))
 //   constant decay:          M <- g M + k v^T;                 o = M^T q                   (g a constant of the head; silu on q, k, v)
 // column j only needs k, q, the token's scalars and v_j.  So a column is owned by LPC lanes of a warp (LPC a power of two), each
-// holding R rows of it in registers for the whole call; tokens are taken in order.  Half of the block's warps own columns; the
-// other half stage the NEXT 16 tokens meanwhile in the second of two shared-memory buffers: their k / q (/ alpha) rows, scalars
+// holding R rows of it in registers for the whole call; tokens are taken in order.  A third of the block's warps own columns; the
+// others stage the NEXT 16 tokens meanwhile in the second of two shared-memory buffers: their k / q (/ alpha) rows, scalars
 // and v, with unit norms, decays and gates evaluated there in 32-bit floats.
 // For the delta rule both dot products are taken on the state BEFORE the token's update,
 //   a = M_old^T k,  c = M_old^T q:   u = beta (v - g a),   o = g c + (k . q) u,   M <- g M_old + k u^T,
@@ -69,10 +69,22 @@ __global__ void token_shift_mix_kernel(const T* __restrict__ h, int B, int S, in
 }
 
 constexpr int REC_CONSUMERS = 128;                          // threads that own state columns (4 warps)
-constexpr int REC_PRODUCERS = 128;                          // threads that stage the next tokens meanwhile (4 warps)
+constexpr int REC_TC = 16;                                  // tokens per stage
+constexpr int REC_PRODUCERS = 256;                          // threads that stage the next tokens meanwhile (8 warps)
+constexpr int REC_TPW = REC_TC / (REC_PRODUCERS / 32);      // tokens a producer warp stages at a time
 constexpr int REC_THREADS = REC_CONSUMERS + REC_PRODUCERS;
-constexpr int REC_TPW = 4;                                  // tokens a producer warp stages at a time
-constexpr int REC_TC = REC_TPW * (REC_PRODUCERS / 32);      // tokens per stage (16)
+
+// the state row that register r of a column's lane `sub` holds: groups of four neighbours, so that a lane reads its share of a k, q or
+// decay row as 16-byte words and the lanes of a column read one contiguous run
+__device__ __forceinline__ int rec_row(int r, int lpc, int sub) { return (((r >> 2) * lpc + sub) << 2) + (r & 3); }
+template <int R>
+__device__ __forceinline__ void rec_load_row(float (&dst)[R], const float* __restrict__ row, int lpc, int sub) {
+#pragma unroll
+    for (int j = 0; j < R / 4; ++j) {
+        const float4 v = *reinterpret_cast<const float4*>(row + ((j * lpc + sub) << 2));
+        dst[4 * j] = v.x; dst[4 * j + 1] = v.y; dst[4 * j + 2] = v.z; dst[4 * j + 3] = v.w;
+    }
+}
 
 // which modes stage a row of decays per token (one per key channel) beside k and q
 __host__ __device__ constexpr bool rec_decay_rows(int mode) { return mode == 1 || mode == 2 || mode == 3; }
@@ -242,14 +254,121 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
     }
 }
 
-// MINB: blocks that must fit an SM together.  0 (no demand) leaves the choice of registers to the compiler (a grid of at most
-// one block per SM: what counts is how fast ONE block walks its tokens; demanding 1 explicitly made it take more registers and
-// run 10 % slower); 2 halves them (some spills) so that two blocks hide each other's latencies, which pays when the grid has
-// more blocks than the GPU has SMs (batches, many heads): measured for the wkv mode only.
-template <typename T, int MODE, int R, int MINB>           // MODE 0: gated delta rule, 1: gated linear attention, 2: wkv,
+// consumers: the stage's nt tokens in order; a column's lanes only talk to each other.  Several partial sums per dot product keep the
+// dependent chains short.  o: this column's output of the stage's first token, o_ld apart from token to token.
+// Where the output does not feed back into the state (no delta rule), the tokens' sums over the column's lanes are independent:
+// they are taken eight tokens at a time, each exchange halving the number of tokens a lane still adds up, so that lane t of eight
+// ends with token t's output (7 exchanges for 8 tokens instead of 3 each).
+template <int MODE, int R>
+__device__ __forceinline__ float rec_step(const RecStage<MODE>& st, float (&M)[R], int tt, int dp, int lpc, int sub, float v, float g_const) {
+    float kr[R], qr[R];
+    rec_load_row<R>(kr, st.k + tt * dp, lpc, sub);
+    rec_load_row<R>(qr, st.q + tt * dp, lpc, sub);
+    float op[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    if (MODE == 1 || MODE == 2) {
+        float ar[R];
+        rec_load_row<R>(ar, st.a + tt * dp, lpc, sub);
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            if (MODE == 2) op[r & 3] += M[r] * qr[r];
+            M[r] = ar[r] * M[r] + kr[r] * v;
+            if (MODE == 1) op[r & 3] += M[r] * qr[r];
+        }
+    } else {
+        const float g = MODE == 4 ? st.sc[tt * 4 + 0] : g_const, w = MODE == 4 ? st.sc[tt * 4 + 1] * v : v;
+#pragma unroll
+        for (int r = 0; r < R; ++r) { M[r] = g * M[r] + kr[r] * w; op[r & 3] += M[r] * qr[r]; }
+    }
+    return (op[0] + op[1]) + (op[2] + op[3]);
+}
+
+// what a token's output has beside the read-out of the state
+template <int MODE>
+__device__ __forceinline__ float rec_extra(const RecStage<MODE>& st, int tt, float v, float skip) {
+    return MODE == 2 ? st.sc[tt * 4 + 2] * v : (MODE == 4 ? skip * v : 0.0f);
+}
+
+template <int MODE, int R>
+__device__ __forceinline__ void rec_walk(const RecStage<MODE>& st, float (&M)[R], int nt, int dp, int cols_blk, int lpc, int sub, int col_l, float g_const,
+                                         float skip, float* __restrict__ o, long o_ld, bool col_ok) {
+    const float* vcol = st.v + col_l;
+    if (MODE == 0 || MODE == 3) {
+        float kr[R], qr[R], ar[MODE == 3 ? R : 4];
+        auto load = [&](int tt) {
+            rec_load_row<R>(kr, st.k + tt * dp, lpc, sub);
+            rec_load_row<R>(qr, st.q + tt * dp, lpc, sub);
+            if constexpr (MODE == 3) rec_load_row<R>(ar, st.a + tt * dp, lpc, sub);
+        };
+        for (int tt = 0; tt < nt; ++tt) {
+            load(tt);
+            const float v = vcol[tt * cols_blk];
+            const float4 sc = *reinterpret_cast<const float4*>(st.sc + tt * 4);                   // g, beta, k . q
+            float ak[4] = {0.0f, 0.0f, 0.0f, 0.0f}, cq[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+                if constexpr (MODE == 3) M[r] *= ar[r];
+                ak[r & 3] += M[r] * kr[r];
+                cq[r & 3] += M[r] * qr[r];
+            }
+            float aks = (ak[0] + ak[1]) + (ak[2] + ak[3]), cqs = (cq[0] + cq[1]) + (cq[2] + cq[3]);
+            if (MODE == 0) {
+#pragma unroll
+                for (int r = 0; r < R; ++r) M[r] *= sc.x;                    // overlaps the exchanges below
+            }
+            for (int m = lpc >> 1; m > 0; m >>= 1) { aks += __shfl_xor_sync(0xffffffffu, aks, m); cqs += __shfl_xor_sync(0xffffffffu, cqs, m); }
+            const float u = MODE == 0 ? sc.y * (v - sc.x * aks) : sc.y * (v - aks);
+#pragma unroll
+            for (int r = 0; r < R; ++r) M[r] += kr[r] * u;
+            if (sub == 0 && col_ok) o[tt * o_ld] = (MODE == 0 ? sc.x * cqs : cqs) + sc.z * u;
+        }
+        return;
+    }
+    int tt = 0;
+    for (; tt + 8 <= nt; tt += 8) {
+        float p[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) p[j] = rec_step<MODE, R>(st, M, tt + j, dp, lpc, sub, vcol[(tt + j) * cols_blk], g_const);
+        if (lpc >= 8) {
+            for (int m = lpc >> 1; m >= 8; m >>= 1) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) p[j] += __shfl_xor_sync(0xffffffffu, p[j], m);
+            }
+            const bool b2 = sub & 4, b1 = sub & 2, b0 = sub & 1;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float keep = b2 ? p[j + 4] : p[j], give = b2 ? p[j] : p[j + 4];
+                p[j] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+            }
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const float keep = b1 ? p[j + 2] : p[j], give = b1 ? p[j] : p[j + 2];
+                p[j] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+            }
+            const float keep = b0 ? p[1] : p[0], give = b0 ? p[0] : p[1];
+            const float mine = keep + __shfl_xor_sync(0xffffffffu, give, 1);
+            if (sub < 8 && col_ok) o[(tt + sub) * o_ld] = mine + rec_extra<MODE>(st, tt + sub, vcol[(tt + sub) * cols_blk], skip);
+        } else {
+            for (int m = lpc >> 1; m > 0; m >>= 1) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) p[j] += __shfl_xor_sync(0xffffffffu, p[j], m);
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+                if ((j & (lpc - 1)) == sub && col_ok) o[(tt + j) * o_ld] = p[j] + rec_extra<MODE>(st, tt + j, vcol[(tt + j) * cols_blk], skip);
+        }
+    }
+    for (; tt < nt; ++tt) {
+        const float v = vcol[tt * cols_blk];
+        float sum = rec_step<MODE, R>(st, M, tt, dp, lpc, sub, v, g_const);
+        for (int m = lpc >> 1; m > 0; m >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, m);
+        if (sub == 0 && col_ok) o[tt * o_ld] = sum + rec_extra<MODE>(st, tt, v, skip);
+    }
+}
+
+template <typename T, int MODE, int R>                     // MODE 0: gated delta rule, 1: gated linear attention, 2: wkv,
                                                            // 3: channel delta rule, 4: state-space scan, 5: constant decay
-__global__ void __launch_bounds__(REC_THREADS, MINB) linear_recurrence_kernel(RecArgs a) {
-    extern __shared__ float sh[];
+__global__ void __launch_bounds__(REC_THREADS) linear_recurrence_kernel(RecArgs a) {
+    extern __shared__ __align__(16) float sh[];
     const int lpc = a.lpc, dp = R * lpc, tc = a.tc;
     const int cols_blk = REC_CONSUMERS / lpc;
     const size_t stage_floats = RecStage<MODE>::floats(tc, dp, cols_blk);
@@ -268,7 +387,7 @@ __global__ void __launch_bounds__(REC_THREADS, MINB) linear_recurrence_kernel(Re
     float* stp = a.state + ((long)b * a.heads + h) * dim * vdim;
 #pragma unroll
     for (int r = 0; r < R; ++r) {
-        int i = r * lpc + sub;
+        const int i = rec_row(r, lpc, sub);
         M[r] = (col_ok && i < dim) ? stp[(long)i * vdim + col] : 0.0f;
     }
     int first = a.pad ? a.pad[b] - a.slot0 : 0;
@@ -299,82 +418,16 @@ __global__ void __launch_bounds__(REC_THREADS, MINB) linear_recurrence_kernel(Re
                                           (S - t1 < tc ? S - t1 : tc), dp, cols_blk, col0, tid - REC_CONSUMERS, neg_exp_a, dt_bias);
             }
         } else {
-            // the tokens in order; a column's lanes only talk to each other.  Four partial sums per dot product keep the
-            // dependent chains short.
             const RecStage<MODE> st(sh + (ci & 1) * stage_floats, tc, dp, cols_blk);
-            const int nt = S - t0 < tc ? S - t0 : tc;
-            for (int tt = 0; tt < nt; ++tt) {
-                const float* kk = st.k + tt * dp + sub;
-                const float* qq = st.q + tt * dp + sub;
-                const float v = st.v[tt * cols_blk + col_l];
-                float kr[R], qr[R];
-#pragma unroll
-                for (int r = 0; r < R; ++r) { kr[r] = kk[r * lpc]; qr[r] = qq[r * lpc]; }
-                float o;
-                if (MODE == 0) {
-                    const float g = st.sc[tt * 4 + 0], beta = st.sc[tt * 4 + 1], kq = st.sc[tt * 4 + 2];
-                    float ak[4] = {0.0f, 0.0f, 0.0f, 0.0f}, cq[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-                    for (int r = 0; r < R; ++r) { ak[r & 3] += M[r] * kr[r]; cq[r & 3] += M[r] * qr[r]; }
-                    float aks = (ak[0] + ak[1]) + (ak[2] + ak[3]), cqs = (cq[0] + cq[1]) + (cq[2] + cq[3]);
-#pragma unroll
-                    for (int r = 0; r < R; ++r) M[r] *= g;                   // overlaps the shuffles below
-                    for (int m = lpc >> 1; m > 0; m >>= 1) { aks += __shfl_xor_sync(0xffffffffu, aks, m); cqs += __shfl_xor_sync(0xffffffffu, cqs, m); }
-                    const float u = beta * (v - g * aks);
-                    o = g * cqs + kq * u;
-#pragma unroll
-                    for (int r = 0; r < R; ++r) M[r] += kr[r] * u;
-                } else if (MODE == 3) {
-                    const float* aa = st.a + tt * dp + sub;
-                    const float beta = st.sc[tt * 4 + 1], kq = st.sc[tt * 4 + 2];
-                    float ak[4] = {0.0f, 0.0f, 0.0f, 0.0f}, cq[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-                    for (int r = 0; r < R; ++r) { M[r] *= aa[r * lpc]; ak[r & 3] += M[r] * kr[r]; cq[r & 3] += M[r] * qr[r]; }
-                    float aks = (ak[0] + ak[1]) + (ak[2] + ak[3]), cqs = (cq[0] + cq[1]) + (cq[2] + cq[3]);
-                    for (int m = lpc >> 1; m > 0; m >>= 1) { aks += __shfl_xor_sync(0xffffffffu, aks, m); cqs += __shfl_xor_sync(0xffffffffu, cqs, m); }
-                    const float u = beta * (v - aks);
-                    o = cqs + kq * u;
-#pragma unroll
-                    for (int r = 0; r < R; ++r) M[r] += kr[r] * u;
-                } else if (MODE == 4) {
-                    const float g = st.sc[tt * 4 + 0], dv = st.sc[tt * 4 + 1] * v;
-                    float op[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-                    for (int r = 0; r < R; ++r) { M[r] = g * M[r] + kr[r] * dv; op[r & 3] += M[r] * qr[r]; }
-                    o = (op[0] + op[1]) + (op[2] + op[3]);
-                    for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
-                    o += skip * v;
-                } else if (MODE == 5) {
-                    float op[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-                    for (int r = 0; r < R; ++r) { M[r] = g_const * M[r] + kr[r] * v; op[r & 3] += M[r] * qr[r]; }
-                    o = (op[0] + op[1]) + (op[2] + op[3]);
-                    for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
-                } else if (MODE == 1) {
-                    const float* aa = st.a + tt * dp + sub;
-                    float op[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-                    for (int r = 0; r < R; ++r) { M[r] = aa[r * lpc] * M[r] + kr[r] * v; op[r & 3] += M[r] * qr[r]; }
-                    o = (op[0] + op[1]) + (op[2] + op[3]);
-                    for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
-                } else {
-                    const float* aa = st.a + tt * dp + sub;
-                    float op[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-                    for (int r = 0; r < R; ++r) { op[r & 3] += M[r] * qr[r]; M[r] = aa[r * lpc] * M[r] + kr[r] * v; }
-                    o = (op[0] + op[1]) + (op[2] + op[3]);
-                    for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
-                    o += st.sc[tt * 4 + 2] * v;
-                }
-                if (sub == 0 && col_ok) obase[(long)(t0 + tt) * a.heads * vdim + col] = o;
-            }
+            rec_walk<MODE, R>(st, M, S - t0 < tc ? S - t0 : tc, dp, cols_blk, lpc, sub, col_l, g_const, skip, obase + (long)t0 * a.heads * vdim + col,
+                                    (long)a.heads * vdim, col_ok);
         }
         __syncthreads();
     }
     if (col_ok) {
 #pragma unroll
         for (int r = 0; r < R; ++r) {
-            int i = r * lpc + sub;
+            const int i = rec_row(r, lpc, sub);
             if (i < dim) stp[(long)i * vdim + col] = M[r];
         }
     }
@@ -590,11 +643,9 @@ static int launch_recurrence(RecArgs a, cudaStream_t stream) {
     if (bytes > 160 * 1024) return launch_recurrence_few<T, MODE>(a, stream);  // very wide heads: stages of fewer tokens, unpipelined
     a.lpc = lpc; a.tc = REC_TC;
     dim3 grid((a.vdim + cols_blk - 1) / cols_blk, a.heads, a.B);
-    const bool pair = (MODE == 2 || MODE == 3) && (long)grid.x * grid.y * grid.z > 148 && 2 * bytes <= 200 * 1024;
-    auto kernel = r == 16 ? (pair ? linear_recurrence_kernel<T, MODE, 16, 2> : linear_recurrence_kernel<T, MODE, 16, 0>)
-                          : (pair ? linear_recurrence_kernel<T, MODE, 32, 2> : linear_recurrence_kernel<T, MODE, 32, 0>);
-    static size_t allowed[4] = {48 * 1024, 48 * 1024, 48 * 1024, 48 * 1024};   // per instantiation: raised once, outside any capture
-    size_t& cur = allowed[(r == 16 ? 0 : 1) + (pair ? 2 : 0)];
+    auto kernel = r == 16 ? linear_recurrence_kernel<T, MODE, 16> : linear_recurrence_kernel<T, MODE, 32>;
+    static size_t allowed[2] = {48 * 1024, 48 * 1024};       // per instantiation: raised once, outside any capture
+    size_t& cur = allowed[r == 16 ? 0 : 1];
     if (bytes > cur) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         if (e != cudaSuccess) return (int)e;

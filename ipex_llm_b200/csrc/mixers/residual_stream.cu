@@ -263,6 +263,59 @@ __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, cons
     }
 }
 
+__device__ __forceinline__ void add4(float4& a, float4 b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
+
+// the same without kept streams (no pre_gain, stack, coef) for rows that come in groups of four channels: a thread owns up to K groups
+// and moves each as one word; every load of the row, the norms' weight vectors among them, is issued before its sum of squares
+template <typename T, int K>
+__global__ void sum_residual_norms4_kernel(float* __restrict__ x, int width, const T* __restrict__ y_a, const T* __restrict__ y_c,
+                                           const float* __restrict__ y_b, const float* __restrict__ y_d, float eps, const T* __restrict__ gain1,
+                                           const T* __restrict__ gain2, int gain_vectors, T* __restrict__ h1, T* __restrict__ h2, int replace,
+                                           const T* __restrict__ vec, T* __restrict__ xc, long ld_xc) {
+    __shared__ float red[32];
+    const long base = (long)blockIdx.x * width;
+    float4 v[K], g1[K], g2[K];
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+        const int c = 4 * (threadIdx.x + k * blockDim.x);
+        v[k] = g1[k] = g2[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (c < width) {
+            if (!replace) v[k] = load4(x + base + c);
+            if (y_a) add4(v[k], load4(y_a + base + c));
+            if (y_c) add4(v[k], load4(y_c + base + c));
+            if (y_b) add4(v[k], load4(y_b + base + c));
+            if (y_d) add4(v[k], load4(y_d + base + c));
+            if (vec) add4(v[k], load4(vec + c));
+            if (h1 && gain_vectors) g1[k] = load4(gain1 + c);
+            if (h2 && gain_vectors) g2[k] = load4(gain2 + c);
+        }
+        ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+    }
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+        const int c = 4 * (threadIdx.x + k * blockDim.x);
+        if (c < width) {
+            store4(x + base + c, v[k]);
+            if (xc) store4(xc + (long)blockIdx.x * ld_xc + c, v[k]);
+        }
+    }
+    if (!h1 && !h2) return;
+    const float f = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
+    const float s1 = h1 && !gain_vectors ? to_f(gain1[0]) : 0.0f, s2 = h2 && !gain_vectors ? to_f(gain2[0]) : 0.0f;
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+        const int c = 4 * (threadIdx.x + k * blockDim.x);
+        if (c < width) {
+            const float4 n = make_float4(v[k].x * f, v[k].y * f, v[k].z * f, v[k].w * f);
+            if (h1) store4(h1 + base + c, gain_vectors ? make_float4(n.x * g1[k].x, n.y * g1[k].y, n.z * g1[k].z, n.w * g1[k].w)
+                                                       : make_float4(n.x * s1, n.y * s1, n.z * s1, n.w * s1));
+            if (h2) store4(h2 + base + c, gain_vectors ? make_float4(n.x * g2[k].x, n.y * g2[k].y, n.z * g2[k].z, n.w * g2[k].w)
+                                                       : make_float4(n.x * s2, n.y * s2, n.z * s2, n.w * s2));
+        }
+    }
+}
+
 // out[n, c] = gelu(in[n, c]) with the exact (erf) form
 template <typename T>
 __global__ void gelu_erf_kernel(const T* __restrict__ in, long n, T* __restrict__ out) {
@@ -423,6 +476,20 @@ extern "C" int mixers_sum_residual_norms(int dtype, float* x, long n_rows, int w
                                          const void* vec, void* xc, long ld_xc, mixers_stream_t stream) {
     if (n_rows <= 0) return 0;
     if ((xc && ld_xc < width) || (coef && !stack) || (h1 && !gain1) || (h2 && !gain2)) return (int)cudaErrorInvalidValue;
+    const uintptr_t words = (uintptr_t)x | (uintptr_t)y_b | (uintptr_t)y_d;               // 32-bit rows: 16-byte words
+    const uintptr_t halves = (uintptr_t)y_a | (uintptr_t)y_c | (uintptr_t)vec | (uintptr_t)xc | (uintptr_t)h1 | (uintptr_t)h2 |
+                             (gain_vectors ? (uintptr_t)gain1 | (uintptr_t)gain2 : 0);
+    if (!stack && !coef && !pre_gain && (width & 3) == 0 && width <= 8192 && (words & 15) == 0 && (halves & (dtype == 0 ? 15 : 7)) == 0 &&
+        (!xc || (ld_xc & 3) == 0)) {
+        const int groups = width / 4, one = (groups + 31) / 32 * 32, two = ((groups + 1) / 2 + 31) / 32 * 32;
+#define SN4_LAUNCH(K, TH) MIXERS_DISPATCH(dtype, sum_residual_norms4_kernel<T, K><<<(unsigned)n_rows, TH, 0, (cudaStream_t)stream>>>(                   \
+        x, width, (const T*)y_a, (const T*)y_c, y_b, y_d, eps, (const T*)gain1, (const T*)gain2, gain_vectors, (T*)h1, (T*)h2, replace, (const T*)vec, \
+        (T*)xc, ld_xc))
+        if (one <= 1024 && (n_rows <= 64 || one <= 128)) SN4_LAUNCH(1, one);
+        else SN4_LAUNCH(2, two);
+#undef SN4_LAUNCH
+        return mixers_status();
+    }
     int threads = width > 1024 ? 256 : 128;
     if (n_rows <= 64)                                        // a decoding step's few rows: one round trip to memory for rows up to 8192 wide
         while (threads < 1024 && threads * SN_MAXC < width) threads <<= 1;

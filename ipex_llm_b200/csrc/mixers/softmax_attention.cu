@@ -191,20 +191,18 @@ __global__ void rope_qk_prepare_kernel(const T* __restrict__ proj, int B, int S,
     }
     const int half = rot_dims >> 1;
     const double dpos = (double)pos;
-    for (int c = lane; c < dim; c += 32) {
-        const int r = c - rot_off;
-        float y;
-        if (r >= 0 && r < rot_dims) {
-            const int i = r < half ? r : r - half;
-            double dsn, dcs;
-            sincos(dpos * inv_freq[i], &dsn, &dcs);
-            const float sn = (float)dsn * amp, cs = (float)dcs * amp;
-            const float u = to_f(src[rot_off + i]), v = to_f(src[rot_off + i + half]);
-            y = r < half ? u * cs - v * sn : v * cs + u * sn;
-        } else {
-            y = to_f(src[c]);
-            if (c < ncols) y = y * inv * to_f(k_norm_w[c]);
-        }
+    for (int i = lane; i < half; i += 32) {                 // a rotated pair per lane: its angle is formed once
+        double dsn, dcs;
+        sincos(dpos * inv_freq[i], &dsn, &dcs);
+        const float sn = (float)dsn * amp, cs = (float)dcs * amp;
+        const float u = to_f(src[rot_off + i]), v = to_f(src[rot_off + i + half]);
+        dst[rot_off + i] = from_f<T>(pos >= 0 ? (u * cs - v * sn) * unit : 0.0f);
+        dst[rot_off + i + half] = from_f<T>(pos >= 0 ? (v * cs + u * sn) * unit : 0.0f);
+    }
+    for (int e = lane; e < dim - rot_dims; e += 32) {       // the others, in front of and behind the rotated range
+        const int c = e < rot_off ? e : e + rot_dims;
+        float y = to_f(src[c]);
+        if (c < ncols) y = y * inv * to_f(k_norm_w[c]);
         dst[c] = from_f<T>(pos >= 0 ? y * unit : 0.0f);
     }
 }
