@@ -89,12 +89,23 @@ int mixers_constant_decay_attention(int dtype, const void* proj, int B, int S, i
                                     const float* decay, int act_silu, float* state, int slot0, const int32_t* pad, float* o,
                                     mixers_stream_t stream);
 
+/* Matrix memory of an mLSTM.  proj [B, S, ld]: q, k (heads x dim each), v (heads x vdim) from columns off_q, off_k, off_v; the gates'
+ * logits, one per head, from off_i and off_f.  i = C((proj_i + bias_i)), f = log(sigmoid(C(proj_f + bias_f))), C(z) = cap tanh(z / cap).
+ * Per head, with a running maximum m that starts at 0:  m' = max(f + m, i);  M <- e^(f + m - m') M + e^(i - m') k v^T;  n likewise with k
+ * alone;  o = M^T (q dim^-1/2), below = max(|n . q dim^-1/2|, e^-m') + tiny.  The mixer's read-out is o / below (see
+ * mixers_gated_rms_norm).  Carried in place: state float [B, heads, dim, vdim], norm_state float [B, heads, dim], max_state float
+ * [B, heads, vdim + 1] (m once per column).  o: float [B, S, heads, vdim], below: float [B, S, heads] (0 and 1 for padding). */
+int mixers_mlstm(int dtype, const void* proj, int B, int S, int ld, int off_q, int off_k, int off_v, int off_i, int off_f, int heads, int dim,
+                 int vdim, const void* bias_i, const void* bias_f, float cap, float tiny, float* state, float* norm_state, float* max_state,
+                 int slot0, const int32_t* pad, float* o, float* below, mixers_stream_t stream);
+
 /* out[n, out_col + h * vdim + c] = out_scale * o[n, h, c] / rms(o[n, h, :]) * w[h * w_head_stride + c] * silu(gate[n, off_g + h * vdim + c])
  * (w_head_stride 0: one weight vector [vdim] for every head; vdim: a vector per head, [heads * vdim]).  gate_mode bit 0: the gate
- * is sigmoid(.) instead of silu(.); bit 1: the gate multiplies before the norm, i.e. rms is taken of o * gate. */
+ * is sigmoid(.) instead of silu(.); bit 1: the gate multiplies before the norm, i.e. rms is taken of o * gate.  below (float
+ * [n_rows, heads], may be null): o[n, h, :] is divided by below[n, h] before everything else. */
 int mixers_gated_rms_norm(int dtype, const float* o, long n_rows, int heads, int vdim, const void* gate, int ld_gate, int off_g,
                           const void* w, int w_head_stride, float eps, void* out, int ld_out, int out_col, float out_scale,
-                          int gate_mode, mixers_stream_t stream);
+                          int gate_mode, const float* below, mixers_stream_t stream);
 
 /* o[n, c] *= out_scale * sigmoid(gate[n, off_g + c / per_gate]) in place, o dtype: n_rows rows of cols channels, ld_o apart */
 int mixers_sigmoid_gate(int dtype, void* o, long ld_o, long n_rows, int cols, const void* gate, int ld_gate, int off_g, int per_gate,
@@ -110,11 +121,12 @@ int mixers_rms_pair_sum(int dtype, const void* a, const void* b, const void* w_a
  * as stream `index` and, with coef (dtype [index + 1]), replaced by sum_j coef[j] * stack[j];  h1 = x / rms(x) * gain1[0],
  * h2 = x / rms(x) * gain2[0] in dtype (either may be null).  gain_vectors != 0: gain1 and gain2 are weight vectors [width].
  * replace != 0: x is replaced by the sum of the addends instead of added to (a stream projected anew).  vec (dtype [width], may be
- * null) belongs to the sum.  xc (may be null): the new x in dtype, row n at xc + n * ld_xc. */
+ * null) belongs to the sum.  xc (may be null): the new x in dtype, row n at xc + n * ld_xc.  gain_add is added to every element of
+ * gain1 and gain2 in 32-bit (1 for norms whose weights are stored around zero). */
 int mixers_sum_residual_norms(int dtype, float* x, long n_rows, int width, const void* y_a, const void* y_c, const float* y_b,
                               const float* y_d, const void* pre_gain, float eps, float* stack, long stack_stride, int index,
                               const void* coef, const void* gain1, const void* gain2, int gain_vectors, void* h1, void* h2, int replace,
-                              const void* vec, void* xc, long ld_xc, mixers_stream_t stream);
+                              const void* vec, void* xc, long ld_xc, float gain_add, mixers_stream_t stream);
 
 /* out = exact (erf) gelu of in, n elements */
 int mixers_gelu_erf(int dtype, const void* in, long n, void* out, mixers_stream_t stream);
@@ -161,14 +173,17 @@ int mixers_embed_pair(int dtype, const void* table, float scale, const void* pai
 int mixers_rms_residual(int dtype, float* x, long n_rows, int width, const void* y, int y_is_float, const void* gain, const void* vec,
                         float eps, float* stack, long stack_stride, int index, const void* coef, void* h, mixers_stream_t stream);
 
-/* out = x / rms(x) * gain[0] * vec[:]   (x float, out dtype; gain, vec may be null) */
-int mixers_rms_norm_rows(int dtype, const float* x, long n_rows, int width, const void* gain, const void* vec, float eps, void* out,
-                         mixers_stream_t stream);
+/* out = x / rms(x) * gain[0] * (vec_add + vec[:])   (x float, out dtype; gain, vec may be null) */
+int mixers_rms_norm_rows(int dtype, const float* x, long n_rows, int width, const void* gain, const void* vec, float vec_add, float eps,
+                         void* out, mixers_stream_t stream);
 
 /* xIELU with pq = {p, q}; with a = softplus(p) and c = 1/2 + softplus(q): f(z) = a z^2 + z/2 where z is positive, c (expm1(z) - z) + z/2 elsewhere */
 int mixers_xielu(int dtype, const void* z, long n, const void* pq, void* out, mixers_stream_t stream);
 
-/* out[n, c] = silu(in[n, off_gate + c]) * in[n, off_up + c], c < cols; in: [n_rows, ld] */
+/* out[n * ld_out + c] = act(in[n, off_gate + c]) * in[n, off_up + c], c < cols; in: [n_rows, ld]; act 0 = silu, 1 = the tanh form of gelu */
+int mixers_glu(int dtype, const void* in, long n_rows, int ld, int off_gate, int off_up, int cols, int act, void* out, long ld_out,
+               mixers_stream_t stream);
+/* the same with silu and ld_out = cols */
 int mixers_silu_mul(int dtype, const void* in, long n_rows, int ld, int off_gate, int off_up, int cols, void* out, mixers_stream_t stream);
 
 /* out[n, c] = g' sigmoid(1.702 g') (u' + 1) with g' = min(in[n, off_gate + c], limit), u' = clamp(in[n, off_up + c], -limit, limit) */
@@ -180,7 +195,8 @@ int mixers_gelu_table_mul(int dtype, const void* g, long n_rows, int cols, const
                           void* out, mixers_stream_t stream);
 
 /* RMS norms (plain weights q_w [q_rank], c_w [kv_rank]) of two column ranges of proj [B, S, ld]: columns off_q.. -> cq_out
- * [B * S, q_rank]; columns off_c.. -> store [B, cap, kv_rank] at storage index held + t (zeros for padding).  dyn as above. */
+ * [B * S, q_rank]; columns off_c.. -> store [B, cap, kv_rank] at storage index held + t (zeros for padding).  kv_rank 0: the query
+ * latent alone (store, c_w may be null).  dyn as above. */
 int mixers_latent_prepare(int dtype, const void* proj, int B, int S, int ld, int off_q, int q_rank, const void* q_w, int off_c,
                           int kv_rank, const void* c_w, float eps, void* cq_out, void* store, int cap, int held, int shift,
                           const int32_t* pad, const int32_t* dyn, mixers_stream_t stream);
@@ -196,20 +212,28 @@ int mixers_wide_qkv_prepare(int dtype, const void* proj, int B, int S, int ld, i
                             const void* blend, void* q_out, void* k_store, void* v_store, int cap, int held, int shift,
                             const int32_t* pad, const int32_t* dyn, mixers_stream_t stream);
 
+/* table float [B * S, pairs, 2] = (cos, sin)(position * freq[i]) * amp of every new token (doubles inside; zeros for padding): what the
+ * layers that share these frequencies read instead of forming the angles anew.  held, shift, pad, dyn as in mixers_window_qk_prepare. */
+int mixers_rotary_table(const double* freq, int pairs, float amp, int B, int S, int held, int shift, const int32_t* pad, const int32_t* dyn,
+                        float* table, mixers_stream_t stream);
+
 /* Rotary positions and cache write for the new tokens' queries and keys (columns of proj [B, S, ld]): `heads` query heads of q_dim
  * channels from off_q, `kv_heads` key heads of k_dim channels from off_k and, if vdim > 0, `kv_heads` value heads from off_v.
  * Inside a head channel rot_off + i pairs with rot_off + i + rot_dims / 2: (u, v) -> (u cos a - v sin a, v cos a + u sin a) * amp,
- * a = position * inv_freq[i] (doubles; angle, sine and cosine in double precision).  k_norm_w (may be null): the first
- * k_norm_cols channels of a key head are divided by their root mean square (eps) and multiplied by k_norm_w first.  unit_rms != 0:
+ * a = position * inv_freq[i] (doubles; angle, sine and cosine in double precision).  table (may be null): [B * S, rot_dims / 2, 2] from
+ * mixers_rotary_table, read instead of inv_freq and amp.  v_table (may be null): [B * S, vdim / 2, 2], the values are rotated too, over all
+ * their channels.  flags bit 0: unit_rms (not together with table); bit 1: pairs are channels 2i and 2i + 1 instead of i and i + half.
+ * kv_proj [B, S, ld_kv] (may be null: proj): the buffer whose columns off_k, off_v hold keys and values.  k_norm_w (may be null): the first
+ * k_norm_cols channels of a key head are divided by their root mean square (eps) and multiplied by k_norm_w first.  unit_rms:
  * behind the rotation every query and key head is divided by its root mean square over its channels (eps, no weight); values
  * pass as they are and may be the key columns themselves (off_v = off_k).  q_out dtype
  * [B * S, heads * q_dim]; key of row b, storage index j, head g at k_store + b * k_bs + j * k_ps + g * k_hs (values alike);
  * the new tokens go to index held + t; padding slots store zeros.  dyn as in mixers_window_qk_prepare. */
 int mixers_rope_qk_prepare(int dtype, const void* proj, int B, int S, int ld, int off_q, int off_k, int off_v, int heads, int kv_heads,
                            int q_dim, int k_dim, int vdim, int q_rot_off, int k_rot_off, int rot_dims, const double* inv_freq, float amp,
-                           const void* k_norm_w, int k_norm_cols, float eps, int unit_rms, void* q_out, void* k_store, long k_bs, long k_ps, long k_hs,
-                           void* v_store, long v_bs, long v_ps, long v_hs, int held, int shift, const int32_t* pad, const int32_t* dyn,
-                           mixers_stream_t stream);
+                           const float* table, const float* v_table, int flags, const void* kv_proj, int ld_kv, const void* k_norm_w,
+                           int k_norm_cols, float eps, void* q_out, void* k_store, long k_bs, long k_ps, long k_hs, void* v_store, long v_bs,
+                           long v_ps, long v_hs, int held, int shift, const int32_t* pad, const int32_t* dyn, mixers_stream_t stream);
 
 /* Causal softmax attention of S new tokens per row.  q: head h of token n at q + n * q_ld + h * q_hs.  Key (value) of storage
  * index j, row b, kv head g at k + b * k_bs + j * k_ps + g * k_hs (strides in elements).  The query at storage index c = held
@@ -220,11 +244,15 @@ int mixers_rope_qk_prepare(int dtype, const void* proj, int B, int S, int ld, in
  * allow_tensor_cores: 16-bit models may take the tensor-core kernels: for S >= 16 one block per 64 tokens of a head (head sizes
  * multiples of 16, <= 256); for S <= 16 and at least 4 query heads per kv head one pass over the keys for all heads of a
  * group, the keys split over blocks (dim a multiple of 16, <= 512; vdim 128, 256 or 512), which needs `ws`:
- * mixers_softmax_attention_workspace(...) floats (0: these sizes never take that kernel).  dyn as above. */
+ * mixers_softmax_attention_workspace(...) floats (0: these sizes never take that kernel).  dyn as above.  back (may be null): float
+ * [B * S, vdim / 2, 2], cosine and sine by whose angle every head's output is turned BACK (pair (u, v) -> (u cos + v sin, v cos - u sin))
+ * before it is rounded to dtype: what undoes a rotation of the values.  back_interleaved: pairs are channels 2i, 2i + 1 instead of
+ * i, i + vdim / 2. */
 int mixers_softmax_attention(int dtype, const void* q, long q_ld, long q_hs, const void* k, long k_bs, long k_ps, long k_hs, const void* v,
                              long v_bs, long v_ps, long v_hs, int B, int S, int heads, int kv_heads, int dim, int vdim, int held,
                              int shift, const int32_t* pad, int window, int chunk, float scale, float softcap, const void* sink, void* out,
-                             long ld_out, int out_col, const int32_t* dyn, int allow_tensor_cores, float* ws, mixers_stream_t stream);
+                             long ld_out, int out_col, const int32_t* dyn, int allow_tensor_cores, float* ws, const float* back,
+                             int back_interleaved, mixers_stream_t stream);
 long mixers_softmax_attention_workspace(int dtype, int B, int S, int heads, int kv_heads, int dim, int vdim);
 
 /* Router of a mixture of experts.  z = router h (32-bit; router [n_out, width], h [n_rows, width] in dtype); s = softmax(z) over

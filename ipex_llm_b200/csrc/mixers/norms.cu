@@ -106,11 +106,12 @@ __global__ void __launch_bounds__(LN_THREADS) layer_norm_residual_kernel(float* 
 
 // one warp per (row, head); w_head_stride: 0 = one weight vector [vdim] for every head, vdim = a vector per head [heads * vdim].
 // gate_mode bit 0: the gate is sigmoid(g) instead of silu(g); bit 1: the gate multiplies BEFORE the norm (the root mean square is
-// that of the gated values) instead of after it
+// that of the gated values) instead of after it.  below (may be null): o's head is divided by below[row, head] first (a recurrence
+// that hands on its read-out and its denominator apart).
 template <typename T>
 __global__ void gated_rms_norm_kernel(const float* __restrict__ o, long n_rows, int heads, int vdim, const T* __restrict__ gate, int ld_gate,
                                       int off_g, const T* __restrict__ w, int w_head_stride, float eps, T* __restrict__ out, int ld_out, int out_col,
-                                      float out_scale, int gate_mode) {
+                                      float out_scale, int gate_mode, const float* __restrict__ below) {
     long warp = (blockIdx.x * (long)blockDim.x + threadIdx.x) >> 5;
     int lane = threadIdx.x & 31;
     if (warp >= n_rows * heads) return;
@@ -120,14 +121,15 @@ __global__ void gated_rms_norm_kernel(const float* __restrict__ o, long n_rows, 
     const T* g = gate + n * (long)ld_gate + off_g + h * vdim;
     auto gated = [&](int c) { const float z = to_f(g[c]); return (gate_mode & 1) ? sigmoid_f(z) : silu_f(z); };
     const bool first = (gate_mode & 2) != 0;
+    const float pre = below ? 1.0f / below[warp] : 1.0f;
     float ss = 0.0f;
-    for (int c = lane; c < vdim; c += 32) { float v = first ? src[c] * gated(c) : src[c]; ss += v * v; }
+    for (int c = lane; c < vdim; c += 32) { float v = pre * (first ? src[c] * gated(c) : src[c]); ss += v * v; }
     ss = warp_sum(ss);
     float inv = 1.0f / sqrtf(ss / (float)vdim + eps);
     T* dst = out + n * (long)ld_out + out_col + h * vdim;
     w += (long)h * w_head_stride;
     for (int c = lane; c < vdim; c += 32)
-        dst[c] = from_f<T>(src[c] * inv * to_f(w[c]) * gated(c) * out_scale);
+        dst[c] = from_f<T>(pre * src[c] * inv * to_f(w[c]) * gated(c) * out_scale);
 }
 
 // the same for wide heads (a state-space branch normalises its whole inner width in a few parts): one block per (row, head), the
@@ -146,7 +148,7 @@ __device__ __forceinline__ float gn_block_sum(float v, float* red) {
 template <typename T>
 __global__ void gated_rms_norm_wide_kernel(const float* __restrict__ o, int heads, int vdim, const T* __restrict__ gate, int ld_gate, int off_g,
                                            const T* __restrict__ w, int w_head_stride, float eps, T* __restrict__ out, int ld_out, int out_col,
-                                           float out_scale, int gate_mode) {
+                                           float out_scale, int gate_mode, const float* __restrict__ below) {
     __shared__ float red[32];
     const long item = blockIdx.x;
     const long n = item / heads;
@@ -154,6 +156,7 @@ __global__ void gated_rms_norm_wide_kernel(const float* __restrict__ o, int head
     const float* src = o + item * (long)vdim;
     const T* g = gate + n * (long)ld_gate + off_g + h * vdim;
     const bool first = (gate_mode & 2) != 0;
+    const float pre = below ? 1.0f / below[item] : 1.0f;
     float v[GN_MAXC], gt[GN_MAXC];
     float ss = 0.0f;
 #pragma unroll
@@ -163,7 +166,7 @@ __global__ void gated_rms_norm_wide_kernel(const float* __restrict__ o, int head
         if (c < vdim) {
             const float z = to_f(g[c]);
             gt[k] = (gate_mode & 1) ? sigmoid_f(z) : silu_f(z);
-            v[k] = first ? src[c] * gt[k] : src[c];
+            v[k] = pre * (first ? src[c] * gt[k] : src[c]);
             ss += v[k] * v[k];
         }
     }
@@ -181,7 +184,7 @@ __global__ void gated_rms_norm_wide_kernel(const float* __restrict__ o, int head
 template <typename T, int K>
 __global__ void gated_rms_norm_wide4_kernel(const float* __restrict__ o, int heads, int vdim, const T* __restrict__ gate, int ld_gate, int off_g,
                                             const T* __restrict__ w, int w_head_stride, float eps, T* __restrict__ out, int ld_out, int out_col,
-                                            float out_scale, int gate_mode) {
+                                            float out_scale, int gate_mode, const float* __restrict__ below) {
     __shared__ float red[32];
     const long item = blockIdx.x;
     const long n = item / heads;
@@ -190,6 +193,7 @@ __global__ void gated_rms_norm_wide4_kernel(const float* __restrict__ o, int hea
     const T* g = gate + n * (long)ld_gate + off_g + h * vdim;
     w += (long)h * w_head_stride;
     const bool first = (gate_mode & 2) != 0;
+    const float pre = below ? 1.0f / below[item] : 1.0f;
     auto act = [&](float z) { return (gate_mode & 1) ? sigmoid_f(z) : silu_f(z); };
     float4 v[K], gt[K], wt[K];
 #pragma unroll
@@ -201,6 +205,7 @@ __global__ void gated_rms_norm_wide4_kernel(const float* __restrict__ o, int hea
     float ss = 0.0f;
 #pragma unroll
     for (int k = 0; k < K; ++k) {
+        v[k] = make_float4(pre * v[k].x, pre * v[k].y, pre * v[k].z, pre * v[k].w);
         gt[k] = make_float4(act(gt[k].x), act(gt[k].y), act(gt[k].z), act(gt[k].w));
         const float4 t = make_float4(v[k].x * gt[k].x, v[k].y * gt[k].y, v[k].z * gt[k].z, v[k].w * gt[k].w);
         const float4 u = first ? t : v[k];
@@ -326,7 +331,7 @@ extern "C" int mixers_layer_norm_residual(int dtype, float* x, long n_rows, int 
 
 extern "C" int mixers_gated_rms_norm(int dtype, const float* o, long n_rows, int heads, int vdim, const void* gate, int ld_gate, int off_g,
                                      const void* w, int w_head_stride, float eps, void* out, int ld_out, int out_col, float out_scale,
-                                     int gate_mode, mixers_stream_t stream) {
+                                     int gate_mode, const float* below, mixers_stream_t stream) {
     if (n_rows <= 0) return 0;
     if (gate_mode & ~3) return (int)cudaErrorInvalidValue;
     long warps = n_rows * heads;
@@ -335,7 +340,7 @@ extern "C" int mixers_gated_rms_norm(int dtype, const float* o, long n_rows, int
         ((uintptr_t)o & 15) == 0 && (halves & (dtype == 0 ? 15 : 7)) == 0) {
         const int groups = vdim / 4, one = (groups + 31) / 32 * 32, two = ((groups + 1) / 2 + 31) / 32 * 32;
 #define GN4_LAUNCH(K, TH) MIXERS_DISPATCH(dtype, gated_rms_norm_wide4_kernel<T, K><<<(unsigned)warps, TH, 0, (cudaStream_t)stream>>>( \
-        o, heads, vdim, (const T*)gate, ld_gate, off_g, (const T*)w, w_head_stride, eps, (T*)out, ld_out, out_col, out_scale, gate_mode))
+        o, heads, vdim, (const T*)gate, ld_gate, off_g, (const T*)w, w_head_stride, eps, (T*)out, ld_out, out_col, out_scale, gate_mode, below))
         if (one <= 1024 && (warps <= 64 || one <= 128)) GN4_LAUNCH(1, one);
         else GN4_LAUNCH(2, two);
 #undef GN4_LAUNCH
@@ -348,13 +353,13 @@ extern "C" int mixers_gated_rms_norm(int dtype, const float* o, long n_rows, int
         while (threads < 1024 && threads * GN_MAXC < vdim) threads <<= 1;
         if (warps <= 1024 && threads * 4 <= vdim && threads < 1024) threads <<= 1;   // at least two rounds of loads in flight per thread are enough
         MIXERS_DISPATCH(dtype, gated_rms_norm_wide_kernel<T><<<(unsigned)warps, threads, 0, (cudaStream_t)stream>>>(
-            o, heads, vdim, (const T*)gate, ld_gate, off_g, (const T*)w, w_head_stride, eps, (T*)out, ld_out, out_col, out_scale, gate_mode));
+            o, heads, vdim, (const T*)gate, ld_gate, off_g, (const T*)w, w_head_stride, eps, (T*)out, ld_out, out_col, out_scale, gate_mode, below));
         return mixers_status();
     }
     int blocks = (int)((warps + 3) / 4);
     MIXERS_DISPATCH(dtype, gated_rms_norm_kernel<T><<<blocks, 128, 0, (cudaStream_t)stream>>>(o, n_rows, heads, vdim, (const T*)gate, ld_gate, off_g,
                                                                                                 (const T*)w, w_head_stride, eps, (T*)out, ld_out, out_col,
-                                                                                                out_scale, gate_mode));
+                                                                                                out_scale, gate_mode, below));
     return mixers_status();
 }
 

@@ -8,6 +8,8 @@
 //                                                                                                  per key channel)
 //   state-space scan:        M <- g M + dt k v^T;              o = M^T q + D v            (g = exp(-exp(A) dt), dt = softplus(. + bias))
 //   constant decay:          M <- g M + k v^T;                 o = M^T q                   (g a constant of the head; silu on q, k, v)
+//   mLSTM:                   M <- g M + w k v^T;  n <- g n + w k;  o = M^T q, below = max(|n . q|, exp(-m)) + tiny
+//                            (m <- max(f + m, i), g = exp(f + m_old - m), w = exp(i - m); i, f log gates from capped logits)
 // column j only needs k, q, the token's scalars and v_j.  So a column is owned by LPC lanes of a warp (LPC a power of two), each
 // holding R rows of it in registers for the whole call; tokens are taken in order.  A third of the block's warps own columns; the
 // others stage the NEXT 16 tokens meanwhile in the second of two shared-memory buffers: their k / q (/ alpha) rows, scalars
@@ -17,6 +19,10 @@
 // which is the same arithmetic reordered so that one round of shuffles serves both.
 // The wkv output reads the state BEFORE the token's update plus a bonus for the token itself: o = M_old^T r + (sum_i r_i u_i k_i) v;
 // the bonus factor is a scalar per token and head, formed while the token is staged.
+// The mLSTM's normaliser n is one more column of the state whose "value" is always 1 (column number vdim of a head's vdim + 1); its
+// read-out becomes the token's denominator, which the norm behind the recurrence divides by.  The running maximum m is a chain over
+// the tokens' two scalars: one producer warp walks it while it stages them.  Every block of a head walks its own copy (blocks of a
+// head need not run at the same time), so the stored m has a place per column.
 #include "mixers_common.cuh"
 
 // one block row per token (blockIdx.x), channels across the block and blockIdx.y: no index division in the loop
@@ -105,6 +111,12 @@ struct RecArgs {
     int act_silu;           // constant decay: silu on q, k and v while they are staged
     const void* w0;         // wkv, channel delta: added to the decay logits [heads * dim]
     const void* u;          // wkv: the current token's bonus [heads * dim]; state-space scan: the skip weight D [heads]
+    const void* bias_i;     // mLSTM: added to the input / forget gate's logits (columns off_b / off_a of proj) [heads]
+    const void* bias_f;
+    float cap, tiny;        // mLSTM: the gate logits' cap; added to the denominator
+    float* norm_state;      // mLSTM: n, float [B, heads, dim]
+    float* max_state;       // mLSTM: m, float [B, heads, vdim + 1], the same number for every column
+    float* below;           // mLSTM: the denominators, float [B, S, heads]
     int B, S, heads, dim, vdim, slot0;
     const int32_t* pad;
     float* state;
@@ -114,6 +126,28 @@ struct RecArgs {
 
 // what q, k and v pass on their way into shared memory
 template <int MODE> __device__ __forceinline__ float rec_act(float z, int act_silu) { return MODE == 5 && act_silu ? silu_f(z) : z; }
+
+// columns of the state per head
+template <int MODE> __host__ __device__ __forceinline__ int rec_columns(int vdim) { return vdim + (MODE == 6 ? 1 : 0); }
+
+// mLSTM: lane t < nt of one warp holds token t's gate logits; the running maximum m (the same in every lane) walks over them and each
+// lane leaves its token's {state decay, input weight, exp(-m)} in sc
+template <typename T>
+__device__ __forceinline__ void mlstm_scalars(const RecArgs& a, int h, int nt, int lane, float zi, float zf, float& m, float* __restrict__ sc) {
+    const float li = a.cap * tanhf((zi + to_f(((const T*)a.bias_i)[h])) / a.cap);
+    const float lf = log_sigmoid_f(a.cap * tanhf((zf + to_f(((const T*)a.bias_f)[h])) / a.cap));
+    float before = 0.0f, mine = 0.0f;
+    for (int t = 0; t < nt; ++t) {
+        const float next = fmaxf(__shfl_sync(0xffffffffu, lf, t) + m, __shfl_sync(0xffffffffu, li, t));
+        if (lane == t) { before = m; mine = next; }
+        m = next;
+    }
+    if (lane < nt) {
+        sc[lane * 4 + 0] = expf(lf + before - mine);
+        sc[lane * 4 + 1] = expf(li - mine);
+        sc[lane * 4 + 2] = expf(-mine);
+    }
+}
 
 // shared memory of one stage: k, q (and alpha) rows of tc tokens padded to dp, the block's value columns, three scalars a token
 template <int MODE>
@@ -130,7 +164,7 @@ struct RecStage {
 // before the first use of any: a warp issues in order, so each wait on memory would otherwise be paid in full, ~20 times a stage.
 template <typename T, int MODE>
 __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE> st, int b, int h, int qh, int t0, int nt, int dp, int cols_blk,
-                                                 int col0, int ptid, float neg_exp_a, float dt_bias) {
+                                                 int col0, int ptid, float neg_exp_a, float dt_bias, float& m_run) {
     const int lane = ptid & 31, pw = ptid >> 5;
     const int dim = a.dim, S = a.S;
     const T* src = (const T*)a.src;
@@ -149,6 +183,7 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
         if (i < nv) {
             int tt = i / cols_blk, cg = col0 + (i - tt * cols_blk);
             if (cg < a.vdim) vreg[e] = rec_act<MODE>(to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * a.vdim + cg]), a.act_silu);
+            else if (MODE == 6 && cg == a.vdim) vreg[e] = 1.0f;
         }
     }
     float lb = 0.0f, la = 0.0f;                              // lane j: the gate logits of the warp's token j
@@ -156,6 +191,11 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
         const T* pr = (const T*)a.proj + ((long)b * S + t0 + tt0 + lane) * a.ld_proj;
         if (MODE != 4) lb = to_f(pr[a.off_b + h]);
         if (MODE != 3) la = to_f(pr[a.off_a + h]);
+    }
+    if (MODE == 6 && pw == 0 && lane < nt) {                // the first warp: both logits of every token of the stage
+        const T* pr = (const T*)a.proj + ((long)b * S + t0 + lane) * a.ld_proj;
+        lb = to_f(pr[a.off_b + h]);
+        la = to_f(pr[a.off_a + h]);
     }
     if (cnt > 0) {
         float sq[REC_TPW], sk[REC_TPW], skq[REC_TPW];
@@ -201,6 +241,8 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
                                 skq[j] += qv[j][e] * uv[e] * kv[j][e];
                             } else if (MODE == 4 || MODE == 5) {
                                 st.q[(tt0 + j) * dp + i] = qv[j][e];
+                            } else if (MODE == 6) {
+                                st.q[(tt0 + j) * dp + i] = qv[j][e] * q_scale;
                             } else {
                                 if (MODE == 3) st.a[(tt0 + j) * dp + i] = i < dim ? expf(neg_exp_a * softplus_f(zv[j][e] + w0v[e])) : 1.0f;
                                 st.q[(tt0 + j) * dp + i] = qv[j][e];
@@ -243,6 +285,7 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
             if (lane < cnt) st.sc[(tt0 + lane) * 4 + 2] = mine;
         }
     }
+    if (MODE == 6 && pw == 0) mlstm_scalars<T>(a, h, nt, lane, lb, la, m_run, st.sc);
 #pragma unroll
     for (int e = 0; e < VB; ++e) {
         int i = ptid + e * REC_PRODUCERS;
@@ -250,7 +293,8 @@ __device__ __forceinline__ void rec_stage_tokens(const RecArgs& a, RecStage<MODE
     }
     for (int i = ptid + VB * REC_PRODUCERS; i < nv; i += REC_PRODUCERS) {          // narrow heads only: more columns than one batch
         int tt = i / cols_blk, cg = col0 + (i - tt * cols_blk);
-        st.v[i] = cg < a.vdim ? rec_act<MODE>(to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * a.vdim + cg]), a.act_silu) : 0.0f;
+        st.v[i] = cg < a.vdim ? rec_act<MODE>(to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * a.vdim + cg]), a.act_silu)
+                              : (MODE == 6 && cg == a.vdim ? 1.0f : 0.0f);
     }
 }
 
@@ -275,17 +319,21 @@ __device__ __forceinline__ float rec_step(const RecStage<MODE>& st, float (&M)[R
             if (MODE == 1) op[r & 3] += M[r] * qr[r];
         }
     } else {
-        const float g = MODE == 4 ? st.sc[tt * 4 + 0] : g_const, w = MODE == 4 ? st.sc[tt * 4 + 1] * v : v;
+        const bool gates = MODE == 4 || MODE == 6;
+        const float g = gates ? st.sc[tt * 4 + 0] : g_const, w = gates ? st.sc[tt * 4 + 1] * v : v;
 #pragma unroll
         for (int r = 0; r < R; ++r) { M[r] = g * M[r] + kr[r] * w; op[r & 3] += M[r] * qr[r]; }
     }
     return (op[0] + op[1]) + (op[2] + op[3]);
 }
 
-// what a token's output has beside the read-out of the state
+// a token's output from the read-out of the state (mLSTM: skip != 0 marks the normaliser's column, g_const holds `tiny`)
 template <int MODE>
-__device__ __forceinline__ float rec_extra(const RecStage<MODE>& st, int tt, float v, float skip) {
-    return MODE == 2 ? st.sc[tt * 4 + 2] * v : (MODE == 4 ? skip * v : 0.0f);
+__device__ __forceinline__ float rec_out(float read, const RecStage<MODE>& st, int tt, float v, float skip, float g_const) {
+    if (MODE == 2) return read + st.sc[tt * 4 + 2] * v;
+    if (MODE == 4) return read + skip * v;
+    if (MODE == 6 && skip != 0.0f) return fmaxf(fabsf(read), st.sc[tt * 4 + 2]) + g_const;
+    return read;
 }
 
 template <int MODE, int R>
@@ -346,7 +394,7 @@ __device__ __forceinline__ void rec_walk(const RecStage<MODE>& st, float (&M)[R]
             }
             const float keep = b0 ? p[1] : p[0], give = b0 ? p[0] : p[1];
             const float mine = keep + __shfl_xor_sync(0xffffffffu, give, 1);
-            if (sub < 8 && col_ok) o[(tt + sub) * o_ld] = mine + rec_extra<MODE>(st, tt + sub, vcol[(tt + sub) * cols_blk], skip);
+            if (sub < 8 && col_ok) o[(tt + sub) * o_ld] = rec_out<MODE>(mine, st, tt + sub, vcol[(tt + sub) * cols_blk], skip, g_const);
         } else {
             for (int m = lpc >> 1; m > 0; m >>= 1) {
 #pragma unroll
@@ -354,19 +402,20 @@ __device__ __forceinline__ void rec_walk(const RecStage<MODE>& st, float (&M)[R]
             }
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-                if ((j & (lpc - 1)) == sub && col_ok) o[(tt + j) * o_ld] = p[j] + rec_extra<MODE>(st, tt + j, vcol[(tt + j) * cols_blk], skip);
+                if ((j & (lpc - 1)) == sub && col_ok) o[(tt + j) * o_ld] = rec_out<MODE>(p[j], st, tt + j, vcol[(tt + j) * cols_blk], skip, g_const);
         }
     }
     for (; tt < nt; ++tt) {
         const float v = vcol[tt * cols_blk];
         float sum = rec_step<MODE, R>(st, M, tt, dp, lpc, sub, v, g_const);
         for (int m = lpc >> 1; m > 0; m >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, m);
-        if (sub == 0 && col_ok) o[tt * o_ld] = sum + rec_extra<MODE>(st, tt, v, skip);
+        if (sub == 0 && col_ok) o[tt * o_ld] = rec_out<MODE>(sum, st, tt, v, skip, g_const);
     }
 }
 
 template <typename T, int MODE, int R>                     // MODE 0: gated delta rule, 1: gated linear attention, 2: wkv,
-                                                           // 3: channel delta rule, 4: state-space scan, 5: constant decay
+                                                           // 3: channel delta rule, 4: state-space scan, 5: constant decay,
+                                                           // 6: mLSTM
 __global__ void __launch_bounds__(REC_THREADS) linear_recurrence_kernel(RecArgs a) {
     extern __shared__ __align__(16) float sh[];
     const int lpc = a.lpc, dp = R * lpc, tc = a.tc;
@@ -379,23 +428,27 @@ __global__ void __launch_bounds__(REC_THREADS) linear_recurrence_kernel(RecArgs 
     const int col_l = tid / lpc;
     const int col0 = blockIdx.x * cols_blk;
     const int col = col0 + col_l;
-    const bool col_ok = !producer && col < a.vdim;
     const int dim = a.dim, vdim = a.vdim, S = a.S;
+    const bool col_ok = !producer && col < rec_columns<MODE>(vdim);
+    const bool norm_col = MODE == 6 && !producer && col == vdim;
     const int qh = h / (a.heads / a.q_heads);
 
     float M[R];
-    float* stp = a.state + ((long)b * a.heads + h) * dim * vdim;
+    // this column's rows of the state and its outputs
+    float* stc = norm_col ? a.norm_state + ((long)b * a.heads + h) * dim : a.state + ((long)b * a.heads + h) * dim * vdim + col;
+    const long st_ld = norm_col ? 1 : vdim;
 #pragma unroll
     for (int r = 0; r < R; ++r) {
         const int i = rec_row(r, lpc, sub);
-        M[r] = (col_ok && i < dim) ? stp[(long)i * vdim + col] : 0.0f;
+        M[r] = (col_ok && i < dim) ? stc[i * st_ld] : 0.0f;
     }
     int first = a.pad ? a.pad[b] - a.slot0 : 0;
     if (first < 0) first = 0;
     if (first > S) first = S;
-    float* obase = a.o + (((long)b * S) * a.heads + h) * vdim;
+    float* ocol = norm_col ? a.below + ((long)b * S) * a.heads + h : a.o + (((long)b * S) * a.heads + h) * vdim + col;
+    const long o_ld = norm_col ? a.heads : (long)a.heads * vdim;
     if (sub == 0 && col_ok)
-        for (int t = 0; t < first; ++t) obase[(long)t * a.heads * vdim + col] = 0.0f;
+        for (int t = 0; t < first; ++t) ocol[t * o_ld] = norm_col ? 1.0f : 0.0f;
 
     const int nchunks = (S - first + tc - 1) / tc;
     float neg_exp_a = 0.0f, dt_bias = 0.0f;
@@ -403,11 +456,13 @@ __global__ void __launch_bounds__(REC_THREADS) linear_recurrence_kernel(RecArgs 
         neg_exp_a = -expf(to_f(((const T*)a.A_log)[h]));
         if (MODE != 3) dt_bias = to_f(((const T*)a.dt_bias)[h]);
     }
-    const float skip = (MODE == 4 && !producer) ? to_f(((const T*)a.u)[h]) : 0.0f;
-    const float g_const = MODE == 5 ? a.decay[h] : 0.0f;
+    const float skip = (MODE == 4 && !producer) ? to_f(((const T*)a.u)[h]) : (norm_col ? 1.0f : 0.0f);
+    const float g_const = MODE == 5 ? a.decay[h] : (MODE == 6 ? a.tiny : 0.0f);
+    float* max_col = MODE == 6 ? a.max_state + ((long)b * a.heads + h) * (vdim + 1) + col0 : nullptr;
+    float m_run = MODE == 6 && producer ? max_col[0] : 0.0f;
     if (producer && nchunks > 0)
         rec_stage_tokens<T, MODE>(a, RecStage<MODE>(sh, tc, dp, cols_blk), b, h, qh, first, (S - first < tc ? S - first : tc), dp, cols_blk, col0,
-                                  tid - REC_CONSUMERS, neg_exp_a, dt_bias);
+                                  tid - REC_CONSUMERS, neg_exp_a, dt_bias, m_run);
     __syncthreads();
     for (int ci = 0; ci < nchunks; ++ci) {
         const int t0 = first + ci * tc;
@@ -415,12 +470,11 @@ __global__ void __launch_bounds__(REC_THREADS) linear_recurrence_kernel(RecArgs 
             if (ci + 1 < nchunks) {
                 const int t1 = t0 + tc;
                 rec_stage_tokens<T, MODE>(a, RecStage<MODE>(sh + ((ci + 1) & 1) * stage_floats, tc, dp, cols_blk), b, h, qh, t1,
-                                          (S - t1 < tc ? S - t1 : tc), dp, cols_blk, col0, tid - REC_CONSUMERS, neg_exp_a, dt_bias);
+                                          (S - t1 < tc ? S - t1 : tc), dp, cols_blk, col0, tid - REC_CONSUMERS, neg_exp_a, dt_bias, m_run);
             }
         } else {
             const RecStage<MODE> st(sh + (ci & 1) * stage_floats, tc, dp, cols_blk);
-            rec_walk<MODE, R>(st, M, S - t0 < tc ? S - t0 : tc, dp, cols_blk, lpc, sub, col_l, g_const, skip, obase + (long)t0 * a.heads * vdim + col,
-                                    (long)a.heads * vdim, col_ok);
+            rec_walk<MODE, R>(st, M, S - t0 < tc ? S - t0 : tc, dp, cols_blk, lpc, sub, col_l, g_const, skip, ocol + t0 * o_ld, o_ld, col_ok);
         }
         __syncthreads();
     }
@@ -428,8 +482,11 @@ __global__ void __launch_bounds__(REC_THREADS) linear_recurrence_kernel(RecArgs 
 #pragma unroll
         for (int r = 0; r < R; ++r) {
             const int i = rec_row(r, lpc, sub);
-            if (i < dim) stp[(long)i * vdim + col] = M[r];
+            if (i < dim) stc[i * st_ld] = M[r];
         }
+    }
+    if (MODE == 6 && producer && tid < REC_CONSUMERS + 32) {                 // the warp that walked the maximum, the block's columns
+        for (int c = tid - REC_CONSUMERS; c < cols_blk && col0 + c <= vdim; c += 32) max_col[c] = m_run;
     }
 }
 
@@ -453,24 +510,29 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
     const int sub = tid % lpc;
     const int col_l = tid / lpc;
     const int col = blockIdx.x * cols_blk + col_l;
-    const bool col_ok = col < a.vdim;
     const int dim = a.dim, vdim = a.vdim, S = a.S;
+    const bool col_ok = col < rec_columns<MODE>(vdim);
+    const bool norm_col = MODE == 6 && col == vdim;
     const int qh = h / (a.heads / a.q_heads);
     const T* src = (const T*)a.src;
 
     float M[R];
-    float* st = a.state + ((long)b * a.heads + h) * dim * vdim;
+    float* stc = norm_col ? a.norm_state + ((long)b * a.heads + h) * dim : a.state + ((long)b * a.heads + h) * dim * vdim + col;
+    const long st_ld = norm_col ? 1 : vdim;
 #pragma unroll
     for (int r = 0; r < R; ++r) {
         int i = r * lpc + sub;
-        M[r] = (col_ok && i < dim) ? st[(long)i * vdim + col] : 0.0f;
+        M[r] = (col_ok && i < dim) ? stc[i * st_ld] : 0.0f;
     }
     int first = a.pad ? a.pad[b] - a.slot0 : 0;
     if (first < 0) first = 0;
     if (first > S) first = S;
-    float* obase = a.o + (((long)b * S) * a.heads + h) * vdim;
+    float* ocol = norm_col ? a.below + ((long)b * S) * a.heads + h : a.o + (((long)b * S) * a.heads + h) * vdim + col;
+    const long o_ld = norm_col ? a.heads : (long)a.heads * vdim;
     if (sub == 0 && col_ok)
-        for (int t = 0; t < first; ++t) obase[(long)t * a.heads * vdim + col] = 0.0f;
+        for (int t = 0; t < first; ++t) ocol[t * o_ld] = norm_col ? 1.0f : 0.0f;
+    float* max_col = MODE == 6 ? a.max_state + ((long)b * a.heads + h) * (vdim + 1) + blockIdx.x * cols_blk : nullptr;
+    float m_run = MODE == 6 ? max_col[0] : 0.0f;             // warp 0 walks it
     const float q_scale = rsqrtf((float)dim);
     const float skip = MODE == 4 ? to_f(((const T*)a.u)[h]) : 0.0f;
     const float g_const = MODE == 5 ? a.decay[h] : 0.0f;
@@ -520,6 +582,8 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
                 }
             } else if (MODE == 5) {
                 // nothing but q, k and v
+            } else if (MODE == 6) {
+                for (int i = lane; i < dp; i += 32) qbuf[tt * dp + i] *= q_scale;
             } else if (MODE == 1) {
                 const T* zr = (const T*)a.z + ((long)b * S + t0 + tt) * ((long)a.heads * dim) + h * dim;
                 for (int i = lane; i < dp; i += 32) {
@@ -542,7 +606,17 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
         for (int i = tid; i < nt * cols_blk; i += REC_FEW_THREADS) {
             int tt = i / cols_blk, cl = i - tt * cols_blk;
             int cg = blockIdx.x * cols_blk + cl;
-            vbuf[i] = cg < vdim ? rec_act<MODE>(to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * vdim + cg]), a.act_silu) : 0.0f;
+            vbuf[i] = cg < vdim ? rec_act<MODE>(to_f(src[((long)b * S + t0 + tt) * a.ld_src + a.off_v + h * vdim + cg]), a.act_silu)
+                                : (MODE == 6 && cg == vdim ? 1.0f : 0.0f);
+        }
+        if (MODE == 6 && wid == 0) {
+            float zi = 0.0f, zf = 0.0f;
+            if (lane < nt) {
+                const T* pr = (const T*)a.proj + ((long)b * S + t0 + lane) * a.ld_proj;
+                zi = to_f(pr[a.off_b + h]);
+                zf = to_f(pr[a.off_a + h]);
+            }
+            mlstm_scalars<T>(a, h, nt, lane, zi, zf, m_run, sc);
         }
         __syncthreads();
         // ---- the tokens in order; a column's lanes only talk to each other
@@ -578,6 +652,13 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
                 for (int r = 0; r < R; ++r) { M[r] = g * M[r] + kk[r * lpc] * dv; o += M[r] * qq[r * lpc]; }
                 for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
                 o += skip * v;
+            } else if (MODE == 6) {
+                const float g = sc[tt * 4 + 0], wv = sc[tt * 4 + 1] * v;
+                o = 0.0f;
+#pragma unroll
+                for (int r = 0; r < R; ++r) { M[r] = g * M[r] + kk[r * lpc] * wv; o += M[r] * qq[r * lpc]; }
+                for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
+                if (norm_col) o = fmaxf(fabsf(o), sc[tt * 4 + 2]) + a.tiny;
             } else if (MODE == 5) {
                 o = 0.0f;
 #pragma unroll
@@ -597,16 +678,18 @@ __global__ void __launch_bounds__(REC_FEW_THREADS) linear_recurrence_few_kernel(
                 for (int m = lpc >> 1; m > 0; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
                 o += sc[tt * 4 + 2] * v;
             }
-            if (sub == 0 && col_ok) obase[(long)(t0 + tt) * a.heads * vdim + col] = o;
+            if (sub == 0 && col_ok) ocol[(t0 + tt) * o_ld] = o;
         }
     }
     if (col_ok) {
 #pragma unroll
         for (int r = 0; r < R; ++r) {
             int i = r * lpc + sub;
-            if (i < dim) st[(long)i * vdim + col] = M[r];
+            if (i < dim) stc[i * st_ld] = M[r];
         }
     }
+    if (MODE == 6 && wid == 0)
+        for (int c = lane; c < cols_blk && (int)blockIdx.x * cols_blk + c <= vdim; c += 32) max_col[c] = m_run;
 }
 
 
@@ -624,7 +707,7 @@ static int launch_recurrence_few(RecArgs a, cudaStream_t stream) {
     while (tc > 1 && bytes(tc) > 40 * 1024) tc >>= 1;
     if (bytes(tc) > 48 * 1024) return (int)cudaErrorInvalidValue;
     a.lpc = lpc; a.tc = tc;
-    dim3 grid((a.vdim + cols_blk - 1) / cols_blk, a.heads, a.B);
+    dim3 grid((rec_columns<MODE>(a.vdim) + cols_blk - 1) / cols_blk, a.heads, a.B);
     if (r == 16) linear_recurrence_few_kernel<T, MODE, 16><<<grid, REC_FEW_THREADS, bytes(tc), stream>>>(a);
     else linear_recurrence_few_kernel<T, MODE, 32><<<grid, REC_FEW_THREADS, bytes(tc), stream>>>(a);
     return mixers_status();
@@ -642,7 +725,7 @@ static int launch_recurrence(RecArgs a, cudaStream_t stream) {
     size_t bytes = 2 * RecStage<MODE>::floats(REC_TC, dp, cols_blk) * sizeof(float);      // two stages
     if (bytes > 160 * 1024) return launch_recurrence_few<T, MODE>(a, stream);  // very wide heads: stages of fewer tokens, unpipelined
     a.lpc = lpc; a.tc = REC_TC;
-    dim3 grid((a.vdim + cols_blk - 1) / cols_blk, a.heads, a.B);
+    dim3 grid((rec_columns<MODE>(a.vdim) + cols_blk - 1) / cols_blk, a.heads, a.B);
     auto kernel = r == 16 ? linear_recurrence_kernel<T, MODE, 16> : linear_recurrence_kernel<T, MODE, 32>;
     static size_t allowed[2] = {48 * 1024, 48 * 1024};       // per instantiation: raised once, outside any capture
     size_t& cur = allowed[r == 16 ? 0 : 1];
@@ -758,5 +841,19 @@ extern "C" int mixers_constant_decay_attention(int dtype, const void* proj, int 
     a.decay = decay; a.act_silu = act_silu;
     a.B = B; a.S = S; a.heads = heads; a.dim = dim; a.vdim = vdim; a.slot0 = slot0; a.pad = pad; a.state = state; a.o = o;
     MIXERS_DISPATCH(dtype, return (launch_recurrence<T, 5>(a, (cudaStream_t)stream)));
+    return 0;
+}
+
+extern "C" int mixers_mlstm(int dtype, const void* proj, int B, int S, int ld, int off_q, int off_k, int off_v, int off_i, int off_f, int heads, int dim,
+                            int vdim, const void* bias_i, const void* bias_f, float cap, float tiny, float* state, float* norm_state, float* max_state,
+                            int slot0, const int32_t* pad, float* o, float* below, mixers_stream_t stream) {
+    if (B <= 0 || S <= 0) return 0;
+    if (!(cap > 0.0f) || !bias_i || !bias_f || !norm_state || !max_state || !below) return (int)cudaErrorInvalidValue;
+    RecArgs a = {};
+    a.src = proj; a.ld_src = ld; a.off_q = off_q; a.off_k = off_k; a.off_v = off_v; a.q_heads = heads;
+    a.proj = proj; a.ld_proj = ld; a.off_b = off_i; a.off_a = off_f; a.bias_i = bias_i; a.bias_f = bias_f; a.cap = cap; a.tiny = tiny;
+    a.norm_state = norm_state; a.max_state = max_state; a.below = below;
+    a.B = B; a.S = S; a.heads = heads; a.dim = dim; a.vdim = vdim; a.slot0 = slot0; a.pad = pad; a.state = state; a.o = o;
+    MIXERS_DISPATCH(dtype, return (launch_recurrence<T, 6>(a, (cudaStream_t)stream)));
     return 0;
 }

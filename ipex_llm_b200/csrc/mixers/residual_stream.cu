@@ -144,7 +144,8 @@ __global__ void rms_residual_cached_kernel(float* __restrict__ x, const TY* __re
 //   VEC: gain1 and gain2 are vectors [width] instead of one number each;
 //   replace: the stream is not added to but replaced by the sum of the addends (a stream that is projected anew);
 //   vec [width]: added to the sum (a vector that belongs to a pass over the layers);
-//   xc: the new x in the model's type, rows ld_xc apart (a column range of what the next projection reads).
+//   xc: the new x in the model's type, rows ld_xc apart (a column range of what the next projection reads);
+//   gain_add: added to every gain in 32-bit (1: norms whose weights are stored around zero).
 // CACHED: the row's elements stay in registers (rows up to SN_MAXC x blockDim wide), every load issued before the first reduction.
 constexpr int SN_MAXC = 8;
 template <typename T, bool CACHED, bool VEC>
@@ -152,7 +153,7 @@ __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, cons
                                           const float* __restrict__ y_b, const float* __restrict__ y_d, const T* __restrict__ pre_gain, float eps,
                                           float* __restrict__ stack, long stack_stride, int index, const T* __restrict__ coef,
                                           const T* __restrict__ gain1, const T* __restrict__ gain2, T* __restrict__ h1, T* __restrict__ h2, int replace,
-                                          const T* __restrict__ vec, T* __restrict__ xc, long ld_xc) {
+                                          const T* __restrict__ vec, T* __restrict__ xc, long ld_xc, float gain_add) {
     __shared__ float red[32];
     const long base = (long)blockIdx.x * width;
     const long base_c = (long)blockIdx.x * ld_xc;
@@ -183,8 +184,8 @@ __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, cons
 #pragma unroll
             for (int k = 0; k < SN_MAXC; ++k) {
                 const int c = threadIdx.x + k * blockDim.x;
-                gv1[k % (VEC ? SN_MAXC : 1)] = h1 && c < width ? to_f(gain1[c]) : 0.0f;
-                gv2[k % (VEC ? SN_MAXC : 1)] = h2 && c < width ? to_f(gain2[c]) : 0.0f;
+                gv1[k % (VEC ? SN_MAXC : 1)] = h1 && c < width ? gain_add + to_f(gain1[c]) : 0.0f;
+                gv2[k % (VEC ? SN_MAXC : 1)] = h2 && c < width ? gain_add + to_f(gain2[c]) : 0.0f;
             }
         }
         if (coef) {
@@ -219,7 +220,7 @@ __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, cons
         }
         if (!want) return;
         const float f = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
-        const float f1 = VEC ? f : (h1 ? f * to_f(gain1[0]) : 0.0f), f2 = VEC ? f : (h2 ? f * to_f(gain2[0]) : 0.0f);
+        const float f1 = VEC ? f : (h1 ? f * (gain_add + to_f(gain1[0])) : 0.0f), f2 = VEC ? f : (h2 ? f * (gain_add + to_f(gain2[0])) : 0.0f);
 #pragma unroll
         for (int k = 0; k < SN_MAXC; ++k) {
             const int c = threadIdx.x + k * blockDim.x;
@@ -255,11 +256,11 @@ __global__ void sum_residual_norms_kernel(float* __restrict__ x, int width, cons
         for (int c = threadIdx.x; c < width; c += blockDim.x) xc[base_c + c] = from_f<T>(x[base + c]);
     if (!want) return;
     const float f = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
-    const float f1 = VEC ? f : (h1 ? f * to_f(gain1[0]) : 0.0f), f2 = VEC ? f : (h2 ? f * to_f(gain2[0]) : 0.0f);
+    const float f1 = VEC ? f : (h1 ? f * (gain_add + to_f(gain1[0])) : 0.0f), f2 = VEC ? f : (h2 ? f * (gain_add + to_f(gain2[0])) : 0.0f);
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         const float v = x[base + c];
-        if (h1) h1[base + c] = from_f<T>(v * f1 * (VEC ? to_f(gain1[c]) : 1.0f));
-        if (h2) h2[base + c] = from_f<T>(v * f2 * (VEC ? to_f(gain2[c]) : 1.0f));
+        if (h1) h1[base + c] = from_f<T>(v * f1 * (VEC ? gain_add + to_f(gain1[c]) : 1.0f));
+        if (h2) h2[base + c] = from_f<T>(v * f2 * (VEC ? gain_add + to_f(gain2[c]) : 1.0f));
     }
 }
 
@@ -271,9 +272,10 @@ template <typename T, int K>
 __global__ void sum_residual_norms4_kernel(float* __restrict__ x, int width, const T* __restrict__ y_a, const T* __restrict__ y_c,
                                            const float* __restrict__ y_b, const float* __restrict__ y_d, float eps, const T* __restrict__ gain1,
                                            const T* __restrict__ gain2, int gain_vectors, T* __restrict__ h1, T* __restrict__ h2, int replace,
-                                           const T* __restrict__ vec, T* __restrict__ xc, long ld_xc) {
+                                           const T* __restrict__ vec, T* __restrict__ xc, long ld_xc, float gain_add) {
     __shared__ float red[32];
     const long base = (long)blockIdx.x * width;
+    const float4 more = make_float4(gain_add, gain_add, gain_add, gain_add);
     float4 v[K], g1[K], g2[K];
     float ss = 0.0f;
 #pragma unroll
@@ -287,8 +289,8 @@ __global__ void sum_residual_norms4_kernel(float* __restrict__ x, int width, con
             if (y_b) add4(v[k], load4(y_b + base + c));
             if (y_d) add4(v[k], load4(y_d + base + c));
             if (vec) add4(v[k], load4(vec + c));
-            if (h1 && gain_vectors) g1[k] = load4(gain1 + c);
-            if (h2 && gain_vectors) g2[k] = load4(gain2 + c);
+            if (h1 && gain_vectors) { g1[k] = load4(gain1 + c); add4(g1[k], more); }
+            if (h2 && gain_vectors) { g2[k] = load4(gain2 + c); add4(g2[k], more); }
         }
         ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
     }
@@ -302,7 +304,7 @@ __global__ void sum_residual_norms4_kernel(float* __restrict__ x, int width, con
     }
     if (!h1 && !h2) return;
     const float f = 1.0f / sqrtf(block_sum(ss, red) / (float)width + eps);
-    const float s1 = h1 && !gain_vectors ? to_f(gain1[0]) : 0.0f, s2 = h2 && !gain_vectors ? to_f(gain2[0]) : 0.0f;
+    const float s1 = h1 && !gain_vectors ? gain_add + to_f(gain1[0]) : 0.0f, s2 = h2 && !gain_vectors ? gain_add + to_f(gain2[0]) : 0.0f;
 #pragma unroll
     for (int k = 0; k < K; ++k) {
         const int c = 4 * (threadIdx.x + k * blockDim.x);
@@ -325,10 +327,10 @@ __global__ void gelu_erf_kernel(const T* __restrict__ in, long n, T* __restrict_
     }
 }
 
-// one block per row: out = x / rms(x) * gain * vec
+// one block per row: out = x / rms(x) * gain * (vec_add + vec)
 template <typename T>
 __global__ void rms_norm_rows_kernel(const float* __restrict__ x, const T* __restrict__ gain, const T* __restrict__ vec, float eps, int width,
-                                     T* __restrict__ out) {
+                                     float vec_add, T* __restrict__ out) {
     __shared__ float red[32];
     const long n = blockIdx.x;
     const float* xr = x + n * width;
@@ -337,7 +339,7 @@ __global__ void rms_norm_rows_kernel(const float* __restrict__ x, const T* __res
     ss = block_sum(ss, red);
     float f = 1.0f / sqrtf(ss / (float)width + eps);
     if (gain) f *= to_f(gain[0]);
-    for (int c = threadIdx.x; c < width; c += blockDim.x) out[n * width + c] = from_f<T>(xr[c] * f * (vec ? to_f(vec[c]) : 1.0f));
+    for (int c = threadIdx.x; c < width; c += blockDim.x) out[n * width + c] = from_f<T>(xr[c] * f * (vec ? vec_add + to_f(vec[c]) : 1.0f));
 }
 
 // xIELU, with a = softplus(p) and c = 1/2 + softplus(q): f(z) = a z^2 + z/2 where z is positive, c (expm1(z) - z) + z/2 elsewhere
@@ -350,16 +352,33 @@ __global__ void xielu_kernel(const T* __restrict__ z, long n, const T* __restric
     }
 }
 
-// out[n, c] = silu(in[n, off_gate + c]) * in[n, off_up + c]
-template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ in, long n_rows, int ld, int off_gate, int off_up, int cols, T* __restrict__ out) {
+// out[n, c] = act(in[n, off_gate + c]) * in[n, off_up + c]; ACT 0: silu, 1: the tanh form of gelu.  The latter is z sigmoid(2 y) with y
+// the tanh's argument, since (1 + tanh y) / 2 = 1 / (1 + e^-2y); 16-bit models take the hardware exponential.
+template <typename T, int ACT> __device__ __forceinline__ float glu_act(float z) {
+    const float a = ACT == 0 ? z : 1.5957691216057308f * (z + 0.044715f * z * z * z);
+    if constexpr (sizeof(T) == 2) return __fdividef(z, 1.0f + __expf(fminf(-a, 80.0f)));
+    return z / (1.0f + expf(-a));
+}
+template <typename T, int ACT>
+__global__ void glu_kernel(const T* __restrict__ in, long n_rows, int ld, int off_gate, int off_up, int cols, T* __restrict__ out,
+                           long ld_out) {
     const long total = n_rows * cols;
     for (long i = blockIdx.x * (long)blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
         const long n = i / cols;
         const int c = (int)(i - n * cols);
         const T* r = in + n * ld;
-        out[i] = from_f<T>(silu_f(to_f(r[off_gate + c])) * to_f(r[off_up + c]));
+        out[n * ld_out + c] = from_f<T>(glu_act<T, ACT>(to_f(r[off_gate + c])) * to_f(r[off_up + c]));
     }
+}
+// the same four neighbours a word: a row per blockIdx.x, its columns across the block and blockIdx.y
+template <typename T, int ACT>
+__global__ void glu4_kernel(const T* __restrict__ in, int ld, int off_gate, int off_up, int cols, T* __restrict__ out, long ld_out) {
+    const long n = blockIdx.x;
+    const T* r = in + n * ld;
+    const int c = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+    if (c >= cols) return;
+    const float4 g = load4(r + off_gate + c), u = load4(r + off_up + c);
+    store4(out + n * ld_out + c, make_float4(glu_act<T, ACT>(g.x) * u.x, glu_act<T, ACT>(g.y) * u.y, glu_act<T, ACT>(g.z) * u.z, glu_act<T, ACT>(g.w) * u.w));
 }
 
 // out[n, c] = g' sigmoid(1.702 g') (u' + 1), g' = min(in[n, off_gate + c], limit), u' = clamp(in[n, off_up + c], -limit, limit)
@@ -431,12 +450,12 @@ extern "C" int mixers_rms_residual(int dtype, float* x, long n_rows, int width, 
     return mixers_status();
 }
 
-extern "C" int mixers_rms_norm_rows(int dtype, const float* x, long n_rows, int width, const void* gain, const void* vec, float eps, void* out,
+extern "C" int mixers_rms_norm_rows(int dtype, const float* x, long n_rows, int width, const void* gain, const void* vec, float vec_add, float eps, void* out,
                                     mixers_stream_t stream) {
     if (n_rows <= 0) return 0;
     const int threads = width >= 1024 ? 256 : 128;
     MIXERS_DISPATCH(dtype, rms_norm_rows_kernel<T><<<(unsigned)n_rows, threads, 0, (cudaStream_t)stream>>>(
-        x, (const T*)gain, (const T*)vec, eps, width, (T*)out));
+        x, (const T*)gain, (const T*)vec, eps, width, vec_add, (T*)out));
     return mixers_status();
 }
 
@@ -446,12 +465,30 @@ extern "C" int mixers_xielu(int dtype, const void* z, long n, const void* pq, vo
     return mixers_status();
 }
 
+extern "C" int mixers_glu(int dtype, const void* in, long n_rows, int ld, int off_gate, int off_up, int cols, int act, void* out, long ld_out,
+                          mixers_stream_t stream) {
+    if (n_rows <= 0 || cols <= 0) return 0;
+    if (act < 0 || act > 1 || ld_out < cols) return (int)cudaErrorInvalidValue;
+    if (((ld | off_gate | off_up | cols | ld_out) & 3) == 0 && (((uintptr_t)in | (uintptr_t)out) & (dtype == 0 ? 15 : 7)) == 0) {
+        const int groups = cols / 4, threads = groups >= 256 ? 256 : (groups + 31) / 32 * 32;
+        const dim3 grid((unsigned)n_rows, (groups + threads - 1) / threads);
+#define GLU4_LAUNCH(A) MIXERS_DISPATCH(dtype, glu4_kernel<T, A><<<grid, threads, 0, (cudaStream_t)stream>>>((const T*)in, ld, off_gate, off_up, cols, (T*)out, ld_out))
+        if (act == 0) GLU4_LAUNCH(0);
+        else GLU4_LAUNCH(1);
+#undef GLU4_LAUNCH
+        return mixers_status();
+    }
+#define GLU_LAUNCH(A) MIXERS_DISPATCH(dtype, glu_kernel<T, A><<<grid_for(n_rows * cols), 256, 0, (cudaStream_t)stream>>>( \
+        (const T*)in, n_rows, ld, off_gate, off_up, cols, (T*)out, ld_out))
+    if (act == 0) GLU_LAUNCH(0);
+    else GLU_LAUNCH(1);
+#undef GLU_LAUNCH
+    return mixers_status();
+}
+
 extern "C" int mixers_silu_mul(int dtype, const void* in, long n_rows, int ld, int off_gate, int off_up, int cols, void* out,
                                mixers_stream_t stream) {
-    if (n_rows <= 0 || cols <= 0) return 0;
-    MIXERS_DISPATCH(dtype, silu_mul_kernel<T><<<grid_for(n_rows * cols), 256, 0, (cudaStream_t)stream>>>(
-        (const T*)in, n_rows, ld, off_gate, off_up, cols, (T*)out));
-    return mixers_status();
+    return mixers_glu(dtype, in, n_rows, ld, off_gate, off_up, cols, 0, out, cols, stream);
 }
 
 extern "C" int mixers_gelu_table_mul(int dtype, const void* g, long n_rows, int cols, const void* table, int ld_table, int col0,
@@ -473,7 +510,7 @@ extern "C" int mixers_clamped_glu(int dtype, const void* in, long n_rows, int ld
 extern "C" int mixers_sum_residual_norms(int dtype, float* x, long n_rows, int width, const void* y_a, const void* y_c, const float* y_b,
                                          const float* y_d, const void* pre_gain, float eps, float* stack, long stack_stride, int index,
                                          const void* coef, const void* gain1, const void* gain2, int gain_vectors, void* h1, void* h2, int replace,
-                                         const void* vec, void* xc, long ld_xc, mixers_stream_t stream) {
+                                         const void* vec, void* xc, long ld_xc, float gain_add, mixers_stream_t stream) {
     if (n_rows <= 0) return 0;
     if ((xc && ld_xc < width) || (coef && !stack) || (h1 && !gain1) || (h2 && !gain2)) return (int)cudaErrorInvalidValue;
     const uintptr_t words = (uintptr_t)x | (uintptr_t)y_b | (uintptr_t)y_d;               // 32-bit rows: 16-byte words
@@ -484,7 +521,7 @@ extern "C" int mixers_sum_residual_norms(int dtype, float* x, long n_rows, int w
         const int groups = width / 4, one = (groups + 31) / 32 * 32, two = ((groups + 1) / 2 + 31) / 32 * 32;
 #define SN4_LAUNCH(K, TH) MIXERS_DISPATCH(dtype, sum_residual_norms4_kernel<T, K><<<(unsigned)n_rows, TH, 0, (cudaStream_t)stream>>>(                   \
         x, width, (const T*)y_a, (const T*)y_c, y_b, y_d, eps, (const T*)gain1, (const T*)gain2, gain_vectors, (T*)h1, (T*)h2, replace, (const T*)vec, \
-        (T*)xc, ld_xc))
+        (T*)xc, ld_xc, gain_add))
         if (one <= 1024 && (n_rows <= 64 || one <= 128)) SN4_LAUNCH(1, one);
         else SN4_LAUNCH(2, two);
 #undef SN4_LAUNCH
@@ -497,7 +534,7 @@ extern "C" int mixers_sum_residual_norms(int dtype, float* x, long n_rows, int w
     const bool cached = width <= SN_MAXC * threads && (n_rows <= 1024 || !coef);
 #define SN_LAUNCH(C, V) MIXERS_DISPATCH(dtype, sum_residual_norms_kernel<T, C, V><<<(unsigned)n_rows, threads, 0, (cudaStream_t)stream>>>(              \
         x, width, (const T*)y_a, (const T*)y_c, y_b, y_d, (const T*)pre_gain, eps, stack, stack_stride, index, (const T*)coef, (const T*)gain1, \
-        (const T*)gain2, (T*)h1, (T*)h2, replace, (const T*)vec, (T*)xc, ld_xc))
+        (const T*)gain2, (T*)h1, (T*)h2, replace, (const T*)vec, (T*)xc, ld_xc, gain_add))
     if (cached && gain_vectors) SN_LAUNCH(true, true);
     else if (cached) SN_LAUNCH(true, false);
     else if (gain_vectors) SN_LAUNCH(false, true);

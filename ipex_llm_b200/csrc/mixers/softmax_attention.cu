@@ -8,24 +8,27 @@
 //   An optional window limits how far back a query looks (0 = every earlier position), optional chunks confine a query to the
 //   earlier positions of its own chunk (chunks counted from the row's first token); scores may be soft-capped
 //   (cap * tanh(score / cap)) and the softmax's denominator may hold a per-head sink exp(sink_h) that has no key and no value.
+//   Values may have been rotated by their own position before they entered the cache; with a table of the queries' angles the three
+//   attention kernels turn every head's output back by the query's position before it is rounded and written.
+//   rotary_table: cosine and sine of every (new token, pair), formed once per call in double precision for all layers that share them.
 //   wide_qkv_prepare: RMS norm over a token's WHOLE query projection and whole key projection (all heads at once, one weight per
 //     channel), values optionally blended with another layer's values of the same token; keys and values are appended to the
 //     cache.
 #include "mixers_common.cuh"
 #include <math.h>
 
-// one block of 128 threads per (token, segment): segment 0 = query latent, 1 = key/value latent.  Segments up to 1024 wide are
+// one block of 128 threads per (token, segment): segment 0 = query latent, 1 = key/value latent (segs 1: the query latent alone).  Segments up to 1024 wide are
 // held in registers (one round of loads); wider ones are read twice.
 constexpr int LP_THREADS = 128, LP_MAXC = 8;
 template <typename T>
 __global__ void __launch_bounds__(LP_THREADS) latent_prepare_kernel(
         const T* __restrict__ proj, int B, int S, int ld, int off_q, int q_rank, const T* __restrict__ q_w, int off_c, int kv_rank,
         const T* __restrict__ c_w, float eps, T* __restrict__ cq_out, T* __restrict__ store, int cap, int held, int shift,
-        const int32_t* __restrict__ pad, const int32_t* __restrict__ dyn) {
+        const int32_t* __restrict__ pad, const int32_t* __restrict__ dyn, int segs) {
     __shared__ float red[LP_THREADS / 32];
     if (dyn) held = dyn[0];
-    const long n = blockIdx.x >> 1;
-    const int seg = blockIdx.x & 1;
+    const long n = segs == 2 ? blockIdx.x >> 1 : blockIdx.x;
+    const int seg = segs == 2 ? blockIdx.x & 1 : 0;
     const int b = (int)(n / S), t = (int)(n - (long)b * S);
     const bool real = held + t + shift - pad[b] >= 0;       // padding slots hold zeros
     const int width = seg ? kv_rank : q_rank;
@@ -135,6 +138,21 @@ __global__ void __launch_bounds__(QP_THREADS) wide_qkv_prepare_kernel(
     }
 }
 
+// table[n, i] = (cos, sin)(position(n) * freq[i]) * amp for every new token n (zeros for padding): angle, cosine and sine in double precision
+__global__ void rotary_table_kernel(const double* __restrict__ freq, int pairs, float amp, int B, int S, int held, int shift,
+                                    const int32_t* __restrict__ pad, const int32_t* __restrict__ dyn, float2* __restrict__ table) {
+    if (dyn) held = dyn[0];
+    const long e = blockIdx.x * (long)blockDim.x + threadIdx.x;
+    if (e >= (long)B * S * pairs) return;
+    const long n = e / pairs;
+    const int i = (int)(e - n * pairs);
+    const int b = (int)(n / S), t = (int)(n - (long)b * S);
+    const int pos = held + t + shift - pad[b];
+    double sn, cs;
+    sincos((double)pos * freq[i], &sn, &cs);
+    table[e] = pos >= 0 ? make_float2((float)cs * amp, (float)sn * amp) : make_float2(0.0f, 0.0f);
+}
+
 // Rotary positions on the queries and keys of new tokens, taken from the columns of one projection output, with the cache write
 // of keys and values: one warp per (token, head slot) -- `heads` query heads of q_dim channels, `kv_heads` key heads of k_dim
 // channels and, when vdim > 0, `kv_heads` value heads.  Inside a head, channel rot_off + i is paired with channel
@@ -144,11 +162,15 @@ __global__ void __launch_bounds__(QP_THREADS) wide_qkv_prepare_kernel(
 // shares its cache row with a rotated part).  unit_rms: every query and key head is divided by its root mean square over the head
 // behind the rotation (no weight; a rotation keeps the sum of squares, so it is taken of what comes in, the rotated channels
 // counting amp^2 times).  Keys and values go to storage index held + t of caches given by three strides; off_v may equal off_k
-// (values that are the keys before norm and rotation).
+// (values that are the keys before norm and rotation).  table: the angles from rotary_table_kernel instead of inv_freq and amp;
+// v_table: the values are rotated as well, over all their channels; interleaved: pairs are channels 2i and 2i + 1 instead of i and
+// i + half; kv_proj: the keys and values are columns of another buffer than the queries.
 template <typename T>
 __global__ void rope_qk_prepare_kernel(const T* __restrict__ proj, int B, int S, int ld, int off_q, int off_k, int off_v, int heads, int kv_heads,
                                        int q_dim, int k_dim, int vdim, int q_rot_off, int k_rot_off, int rot_dims, const double* __restrict__ inv_freq,
-                                       float amp, const T* __restrict__ k_norm_w, int k_norm_cols, float eps, int unit_rms, T* __restrict__ q_out,
+                                       float amp, const float2* __restrict__ table, const float2* __restrict__ v_table, int interleaved,
+                                       const T* __restrict__ kv_proj, int ld_kv, const T* __restrict__ k_norm_w, int k_norm_cols, float eps, int unit_rms,
+                                       T* __restrict__ q_out,
                                        T* __restrict__ k_store, long k_bs, long k_ps, long k_hs, T* __restrict__ v_store, long v_bs, long v_ps,
                                        long v_hs, int held, int shift, const int32_t* __restrict__ pad, const int32_t* __restrict__ dyn) {
     if (dyn) held = dyn[0];
@@ -160,11 +182,22 @@ __global__ void rope_qk_prepare_kernel(const T* __restrict__ proj, int B, int S,
     const int hs = (int)(warp - n * slots);
     const int b = (int)(n / S), t = (int)(n - (long)b * S);
     const int pos = held + t + shift - pad[b];              // negative: a padding slot
-    const T* row = proj + n * (long)ld;
+    const T* row = hs < heads ? proj + n * (long)ld : kv_proj + n * (long)ld_kv;
     if (hs >= heads + kv_heads) {
         const int g = hs - heads - kv_heads;
         const T* src = row + off_v + g * vdim;
         T* dst = v_store + b * v_bs + (long)(held + t) * v_ps + g * v_hs;
+        if (v_table) {
+            const int vhalf = vdim >> 1;
+            for (int i = lane; i < vhalf; i += 32) {
+                const float2 cs = v_table[n * vhalf + i];
+                const int c0 = interleaved ? 2 * i : i, c1 = interleaved ? 2 * i + 1 : i + vhalf;
+                const float u = to_f(src[c0]), v = to_f(src[c1]);
+                dst[c0] = from_f<T>(pos >= 0 ? u * cs.x - v * cs.y : 0.0f);
+                dst[c1] = from_f<T>(pos >= 0 ? v * cs.x + u * cs.y : 0.0f);
+            }
+            return;
+        }
         for (int c = lane; c < vdim; c += 32) dst[c] = pos >= 0 ? src[c] : from_f<T>(0.0f);
         return;
     }
@@ -192,12 +225,19 @@ __global__ void rope_qk_prepare_kernel(const T* __restrict__ proj, int B, int S,
     const int half = rot_dims >> 1;
     const double dpos = (double)pos;
     for (int i = lane; i < half; i += 32) {                 // a rotated pair per lane: its angle is formed once
-        double dsn, dcs;
-        sincos(dpos * inv_freq[i], &dsn, &dcs);
-        const float sn = (float)dsn * amp, cs = (float)dcs * amp;
-        const float u = to_f(src[rot_off + i]), v = to_f(src[rot_off + i + half]);
-        dst[rot_off + i] = from_f<T>(pos >= 0 ? (u * cs - v * sn) * unit : 0.0f);
-        dst[rot_off + i + half] = from_f<T>(pos >= 0 ? (v * cs + u * sn) * unit : 0.0f);
+        float sn, cs;
+        if (table) {
+            const float2 a = table[n * half + i];
+            cs = a.x; sn = a.y;
+        } else {
+            double dsn, dcs;
+            sincos(dpos * inv_freq[i], &dsn, &dcs);
+            sn = (float)dsn * amp; cs = (float)dcs * amp;
+        }
+        const int c0 = rot_off + (interleaved ? 2 * i : i), c1 = rot_off + (interleaved ? 2 * i + 1 : i + half);
+        const float u = to_f(src[c0]), v = to_f(src[c1]);
+        dst[c0] = from_f<T>(pos >= 0 ? (u * cs - v * sn) * unit : 0.0f);
+        dst[c1] = from_f<T>(pos >= 0 ? (v * cs + u * sn) * unit : 0.0f);
     }
     for (int e = lane; e < dim - rot_dims; e += 32) {       // the others, in front of and behind the rotated range
         const int c = e < rot_off ? e : e + rot_dims;
@@ -206,6 +246,9 @@ __global__ void rope_qk_prepare_kernel(const T* __restrict__ proj, int B, int S,
         dst[c] = from_f<T>(pos >= 0 ? y * unit : 0.0f);
     }
 }
+
+// a pair (u, v) turned by minus the angle whose cosine and sine are a
+__device__ __forceinline__ float2 turn_back(float u, float v, float2 a) { return make_float2(u * a.x + v * a.y, v * a.x - u * a.y); }
 
 // ---- the general kernel: any sizes and strides, any dtype, 32-bit arithmetic throughout (float32 models, decoding, short
 // portions).  A block of SA_WARPS warps per (token, query head); the warps take the visible keys in turns of 32, each with its
@@ -225,13 +268,15 @@ template <typename T>
 __global__ void __launch_bounds__(SA_WARPS * 32) softmax_attention_kernel(
         const T* __restrict__ q, long q_ld, long q_hs, const T* __restrict__ k, long k_bs, long k_ps, long k_hs, const T* __restrict__ v, long v_bs, long v_ps,
         long v_hs, int B, int S, int heads, int kv_heads, int dim, int vdim, int held, int shift, const int32_t* __restrict__ pad, int window, int chunk,
-        float scale, float softcap, const T* __restrict__ sink, T* __restrict__ out, long ld_out, int out_col, const int32_t* __restrict__ dyn, int aligned) {
+        float scale, float softcap, const T* __restrict__ sink, T* __restrict__ out, long ld_out, int out_col, const int32_t* __restrict__ dyn, int aligned,
+        const float2* __restrict__ back, int back_interleaved) {
     extern __shared__ __align__(16) float sa_sh[];          // q [dim rounded up to 4], warp maxima, warp sums, partial values
     const int dim4 = (dim + 3) & ~3;
     float* qs = sa_sh;
     float* wm = sa_sh + dim4;
     float* wl = wm + SA_WARPS;
     float* part = wl + SA_WARPS;                            // [SA_WARPS][SA_VCOLS * 32]
+    float* whole = part + SA_WARPS * SA_VCOLS * 32;         // [vdim], only there when the output is turned back
     if (dyn) held = dyn[0];
     const int wid = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long item = blockIdx.x;
@@ -299,10 +344,21 @@ __global__ void __launch_bounds__(SA_WARPS * 32) softmax_attention_kernel(
                 float sum = 0.0f;
 #pragma unroll
                 for (int w = 0; w < SA_WARPS; ++w) sum += part[w * SA_VCOLS * 32 + e] * f[w];
-                dst[col] = from_f<T>(sum / total);
+                if (back) whole[col] = sum / total;
+                else dst[col] = from_f<T>(sum / total);
             }
         }
         __syncthreads();
+    }
+    if (back) {
+        const int half = vdim >> 1;
+        for (int i = threadIdx.x; i < half; i += blockDim.x) {
+            const float2 a = back[n * half + i];
+            const int c0 = back_interleaved ? 2 * i : i, c1 = back_interleaved ? 2 * i + 1 : i + half;
+            const float2 y = turn_back(whole[c0], whole[c1], a);
+            dst[c0] = from_f<T>(y.x);
+            dst[c1] = from_f<T>(y.y);
+        }
     }
 }
 
@@ -348,7 +404,8 @@ template <typename T, int KDMAX, int NDMAX>                // dim <= 16 KDMAX, v
 __global__ void __launch_bounds__(128) softmax_attention_tc_kernel(
         const T* __restrict__ q, long q_ld, long q_hs, const T* __restrict__ k, long k_bs, long k_ps, long k_hs, const T* __restrict__ v, long v_bs, long v_ps,
         long v_hs, int B, int S, int heads, int kv_heads, int dim, int vdim, int held, int shift, const int32_t* __restrict__ pad, int window, int chunk,
-        float scale, float softcap, const T* __restrict__ sink, T* __restrict__ out, long ld_out, int out_col) {
+        float scale, float softcap, const T* __restrict__ sink, T* __restrict__ out, long ld_out, int out_col, const float2* __restrict__ back,
+        int back_interleaved) {
     extern __shared__ __align__(16) unsigned char sa_tc_sh[];
     const int kstride = dim + 8, vstride = vdim + 8;        // elements
     T* Ks = reinterpret_cast<T*>(sa_tc_sh);                 // two stages of [SA_KEYS][kstride] keys + [SA_KEYS][vstride] values
@@ -522,6 +579,34 @@ __global__ void __launch_bounds__(128) softmax_attention_tc_kernel(
         const float inv = l > 0.0f ? 1.0f / l : 0.0f;
         if (tr[i] < S) {
             T* dst = out + ((long)b * S + tr[i]) * ld_out + out_col + (long)h * vdim + 2 * tq;
+            if (back) {                                     // both channels of a pair are in this thread, whatever the layout
+                const int half = vdim >> 1, nh = ndn >> 1;
+                const float2* angle = back + ((long)b * S + tr[i]) * half;
+                if (back_interleaved) {
+#pragma unroll
+                    for (int nd = 0; nd < NDMAX; ++nd) {
+                        if (nd < ndn) {
+                            const float2 y = turn_back(oacc[nd][2 * i], oacc[nd][2 * i + 1], angle[nd * 4 + tq]);
+                            oacc[nd][2 * i] = y.x;
+                            oacc[nd][2 * i + 1] = y.y;
+                        }
+                    }
+                } else {
+#pragma unroll
+                    for (int nhc = 1; nhc <= NDMAX / 2; ++nhc) {            // the partner tile is nh further: registers need constant indices
+                        if (nhc == nh) {
+#pragma unroll
+                            for (int nd = 0; nd < nhc; ++nd) {
+                                const float4 a = *reinterpret_cast<const float4*>(angle + nd * 8 + 2 * tq);
+                                const float2 y0 = turn_back(oacc[nd][2 * i], oacc[nd + nhc][2 * i], make_float2(a.x, a.y));
+                                const float2 y1 = turn_back(oacc[nd][2 * i + 1], oacc[nd + nhc][2 * i + 1], make_float2(a.z, a.w));
+                                oacc[nd][2 * i] = y0.x; oacc[nd + nhc][2 * i] = y0.y;
+                                oacc[nd][2 * i + 1] = y1.x; oacc[nd + nhc][2 * i + 1] = y1.y;
+                            }
+                        }
+                    }
+                }
+            }
 #pragma unroll
             for (int nd = 0; nd < NDMAX; ++nd) {
                 if (nd < ndn) {
@@ -744,7 +829,8 @@ __global__ void __launch_bounds__(256) shared_head_attention_kernel(
 // maxima into factors; then every thread owns two neighbouring columns and reads them from all ranges (independent loads).
 template <typename T>
 __global__ void __launch_bounds__(256) shared_head_merge_kernel(const float* __restrict__ ws, int S, int heads, int kv_heads, int vdim, int splits,
-                                                                int tiles, const T* __restrict__ sink, T* __restrict__ out, long ld_out, int out_col) {
+                                                                int tiles, const T* __restrict__ sink, T* __restrict__ out, long ld_out, int out_col,
+                                                                const float2* __restrict__ back, int back_interleaved) {
     __shared__ float factor[SH_MAX_SPLITS];
     __shared__ float inv_total;
     const int y = blockIdx.x >> 4, i = blockIdx.x & 15, lane = threadIdx.x & 31;
@@ -766,6 +852,25 @@ __global__ void __launch_bounds__(256) shared_head_merge_kernel(const float* __r
     }
     __syncthreads();
     T* dst = out + ((long)b * S + r / gs) * ld_out + out_col + (long)(g * gs + r % gs) * vdim;
+    if (back) {                                             // a thread owns the two columns of a rotated pair
+        const int half = vdim >> 1;
+        for (int p = threadIdx.x; p < half; p += 256) {
+            const int c0 = back_interleaved ? 2 * p : p, c1 = back_interleaved ? 2 * p + 1 : p + half;
+            const float2 a = back[((long)b * S + r / gs) * half + p];
+            float s0 = 0.0f, s1 = 0.0f;
+#pragma unroll 8
+            for (int s = 0; s < splits; ++s) {
+                if (factor[s] == 0.0f) continue;
+                const float* o = base + s * sstride + 2;
+                s0 += o[c0] * factor[s];
+                s1 += o[c1] * factor[s];
+            }
+            const float2 y = turn_back(s0 * inv_total, s1 * inv_total, a);
+            dst[c0] = from_f<T>(y.x);
+            dst[c1] = from_f<T>(y.y);
+        }
+        return;
+    }
     for (int col = 2 * threadIdx.x; col < vdim; col += 512) {
         float sx = 0.0f, sy = 0.0f;
 #pragma unroll 8
@@ -800,7 +905,8 @@ static size_t shared_head_smem(int dim, int vdim, bool same) {
 template <typename T, int NT>
 static int launch_shared_head(const void* q, long q_ld, long q_hs, const void* k, long k_bs, long k_ps, long k_hs, const void* v, long v_bs, long v_ps, long v_hs,
                               int B, int S, int heads, int kv_heads, int dim, int held, int shift, const int32_t* pad, int window, int chunk, float scale,
-                              float softcap, const void* sink, void* out, long ld_out, int out_col, const int32_t* dyn, float* ws, cudaStream_t stream) {
+                              float softcap, const void* sink, void* out, long ld_out, int out_col, const int32_t* dyn, float* ws, const float2* back,
+                              int back_interleaved, cudaStream_t stream) {
     const int vdim = 64 * NT;
     const int tiles = (S * (heads / kv_heads) + 15) / 16, splits = shared_head_splits(B, S, heads, kv_heads);
     const bool same = k == v && k_bs == v_bs && k_ps == v_ps && k_hs == v_hs && dim >= vdim;     // the values are the keys' first channels
@@ -819,15 +925,16 @@ static int launch_shared_head(const void* q, long q_ld, long q_hs, const void* k
                                         shift, pad, window, chunk, scale, softcap, ws, splits, tiles, dyn);
     }
     if ((err = cudaGetLastError()) != cudaSuccess) return (int)err;
-    shared_head_merge_kernel<T><<<dim3(16 * tiles * kv_heads, B), 256, 0, stream>>>(ws, S, heads, kv_heads, vdim, splits, tiles, (const T*)sink, (T*)out, ld_out, out_col);
+    shared_head_merge_kernel<T><<<dim3(16 * tiles * kv_heads, B), 256, 0, stream>>>(ws, S, heads, kv_heads, vdim, splits, tiles, (const T*)sink, (T*)out, ld_out, out_col,
+                                                                                  back, back_interleaved);
     return mixers_status();
 }
 
 #define SA_TC_PARAMS const void* q, long q_ld, long q_hs, const void* k, long k_bs, long k_ps, long k_hs, const void* v, long v_bs, long v_ps, long v_hs, \
     int B, int S, int heads, int kv_heads, int dim, int vdim, int held, int shift, const int32_t* pad, int window, int chunk, float scale, float softcap,  \
-    const void* sink, void* out, long ld_out, int out_col, cudaStream_t stream
+    const void* sink, void* out, long ld_out, int out_col, const float2* back, int back_interleaved, cudaStream_t stream
 #define SA_TC_ARGS q, q_ld, q_hs, k, k_bs, k_ps, k_hs, v, v_bs, v_ps, v_hs, B, S, heads, kv_heads, dim, vdim, held, shift, pad, window, chunk, scale, softcap, \
-    sink, out, ld_out, out_col, stream
+    sink, out, ld_out, out_col, back, back_interleaved, stream
 
 template <typename T, int KDMAX, int NDMAX>
 static int launch_softmax_tc(SA_TC_PARAMS) {
@@ -839,7 +946,7 @@ static int launch_softmax_tc(SA_TC_PARAMS) {
     }
     softmax_attention_tc_kernel<T, KDMAX, NDMAX><<<grid, 128, smem, stream>>>(
         (const T*)q, q_ld, q_hs, (const T*)k, k_bs, k_ps, k_hs, (const T*)v, v_bs, v_ps, v_hs, B, S, heads, kv_heads, dim, vdim, held, shift, pad, window, chunk,
-        scale, softcap, (const T*)sink, (T*)out, ld_out, out_col);
+        scale, softcap, (const T*)sink, (T*)out, ld_out, out_col, back, back_interleaved);
     return mixers_status();
 }
 
@@ -854,9 +961,10 @@ extern "C" int mixers_latent_prepare(int dtype, const void* proj, int B, int S, 
                                      int kv_rank, const void* c_w, float eps, void* cq_out, void* store, int cap, int held, int shift,
                                      const int32_t* pad, const int32_t* dyn, mixers_stream_t stream) {
     if (B <= 0 || S <= 0) return 0;
-    if (held + S > cap) return (int)cudaErrorInvalidValue;
-    MIXERS_DISPATCH(dtype, latent_prepare_kernel<T><<<(unsigned)(2L * B * S), LP_THREADS, 0, (cudaStream_t)stream>>>(
-        (const T*)proj, B, S, ld, off_q, q_rank, (const T*)q_w, off_c, kv_rank, (const T*)c_w, eps, (T*)cq_out, (T*)store, cap, held, shift, pad, dyn));
+    if (kv_rank > 0 && held + S > cap) return (int)cudaErrorInvalidValue;
+    const int segs = kv_rank > 0 ? 2 : 1;
+    MIXERS_DISPATCH(dtype, latent_prepare_kernel<T><<<(unsigned)((long)segs * B * S), LP_THREADS, 0, (cudaStream_t)stream>>>(
+        (const T*)proj, B, S, ld, off_q, q_rank, (const T*)q_w, off_c, kv_rank, (const T*)c_w, eps, (T*)cq_out, (T*)store, cap, held, shift, pad, dyn, segs));
     return mixers_status();
 }
 
@@ -880,31 +988,44 @@ extern "C" int mixers_wide_qkv_prepare(int dtype, const void* proj, int B, int S
     return mixers_status();
 }
 
+extern "C" int mixers_rotary_table(const double* freq, int pairs, float amp, int B, int S, int held, int shift, const int32_t* pad, const int32_t* dyn,
+                                   float* table, mixers_stream_t stream) {
+    const long total = (long)B * S * pairs;
+    if (total <= 0) return 0;
+    rotary_table_kernel<<<(unsigned)((total + 127) / 128), 128, 0, (cudaStream_t)stream>>>(freq, pairs, amp, B, S, held, shift, pad, dyn, (float2*)table);
+    return mixers_status();
+}
+
 extern "C" int mixers_rope_qk_prepare(int dtype, const void* proj, int B, int S, int ld, int off_q, int off_k, int off_v, int heads, int kv_heads,
                                       int q_dim, int k_dim, int vdim, int q_rot_off, int k_rot_off, int rot_dims, const double* inv_freq, float amp,
-                                      const void* k_norm_w, int k_norm_cols, float eps, int unit_rms, void* q_out, void* k_store, long k_bs, long k_ps,
-                                      long k_hs, void* v_store, long v_bs, long v_ps, long v_hs, int held, int shift, const int32_t* pad,
-                                      const int32_t* dyn, mixers_stream_t stream) {
+                                      const float* table, const float* v_table, int flags, const void* kv_proj, int ld_kv, const void* k_norm_w,
+                                      int k_norm_cols, float eps, void* q_out, void* k_store, long k_bs, long k_ps, long k_hs, void* v_store, long v_bs,
+                                      long v_ps, long v_hs, int held, int shift, const int32_t* pad, const int32_t* dyn, mixers_stream_t stream) {
     if (B <= 0 || S <= 0) return 0;
     if (rot_dims < 0 || (rot_dims & 1) || q_rot_off < 0 || k_rot_off < 0 || q_rot_off + rot_dims > q_dim || k_rot_off + rot_dims > k_dim ||
-        kv_heads < 1 || heads < 1 || (rot_dims > 0 && !inv_freq) || (k_norm_w && (k_norm_cols < 1 || k_norm_cols > k_rot_off)) || (vdim > 0 && !v_store))
+        kv_heads < 1 || heads < 1 || (rot_dims > 0 && !inv_freq && !table) || (k_norm_w && (k_norm_cols < 1 || k_norm_cols > k_rot_off)) ||
+        (vdim > 0 && !v_store) || (flags & ~3) || (v_table && (vdim & 1)) || ((flags & 1) && table))
         return (int)cudaErrorInvalidValue;
     const long warps = (long)B * S * (heads + kv_heads + (vdim > 0 ? kv_heads : 0));
     const unsigned blocks = (unsigned)((warps + 3) / 4);
     MIXERS_DISPATCH(dtype, rope_qk_prepare_kernel<T><<<blocks, 128, 0, (cudaStream_t)stream>>>(
         (const T*)proj, B, S, ld, off_q, off_k, off_v, heads, kv_heads, q_dim, k_dim, vdim, q_rot_off, k_rot_off, rot_dims, inv_freq, amp,
-        (const T*)k_norm_w, k_norm_cols, eps, unit_rms, (T*)q_out, (T*)k_store, k_bs, k_ps, k_hs, (T*)v_store, v_bs, v_ps, v_hs, held, shift, pad, dyn));
+        (const float2*)table, (const float2*)v_table, flags >> 1, (const T*)(kv_proj ? kv_proj : proj), kv_proj ? ld_kv : ld, (const T*)k_norm_w,
+        k_norm_cols, eps, flags & 1, (T*)q_out, (T*)k_store, k_bs, k_ps, k_hs, (T*)v_store, v_bs, v_ps, v_hs, held, shift, pad, dyn));
     return mixers_status();
 }
 
 extern "C" int mixers_softmax_attention(int dtype, const void* q, long q_ld, long q_hs, const void* k, long k_bs, long k_ps, long k_hs, const void* v,
                                         long v_bs, long v_ps, long v_hs, int B, int S, int heads, int kv_heads, int dim, int vdim, int held,
                                         int shift, const int32_t* pad, int window, int chunk, float scale, float softcap, const void* sink, void* out,
-                                        long ld_out, int out_col, const int32_t* dyn, int allow_tensor_cores, float* ws, mixers_stream_t stream_) {
+                                        long ld_out, int out_col, const int32_t* dyn, int allow_tensor_cores, float* ws, const float* back_, int back_interleaved,
+                                        mixers_stream_t stream_) {
     if (B <= 0 || S <= 0) return 0;
     cudaStream_t stream = (cudaStream_t)stream_;
     const int dim4 = (dim + 3) & ~3;
-    size_t smem = ((size_t)dim4 + 2 * SA_WARPS + SA_WARPS * SA_VCOLS * 32) * sizeof(float);
+    const float2* back = (const float2*)back_;
+    size_t smem = ((size_t)dim4 + 2 * SA_WARPS + SA_WARPS * SA_VCOLS * 32 + (back ? vdim : 0)) * sizeof(float);
+    if (back && (vdim & 1)) return (int)cudaErrorInvalidValue;
     if (window < 0 || chunk < 0 || kv_heads < 1 || heads % kv_heads != 0 || smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     const size_t esz = dtype == 0 ? 4 : 2;
     auto mult8 = [](long s) { return (s & 7) == 0; };
@@ -913,7 +1034,7 @@ extern "C" int mixers_softmax_attention(int dtype, const void* q, long q_ld, lon
     const bool same_kv = k == v && k_bs == v_bs && k_ps == v_ps && k_hs == v_hs && dim >= vdim;
     if (allow_tensor_cores && ws && rows16 && shared_head_ok(dtype, S, heads, kv_heads, dim, vdim) && (q_ld & 7) == 0 && (q_hs & 7) == 0 && ((uintptr_t)q & 15) == 0 &&
         (ld_out & 1) == 0 && (out_col & 1) == 0 && shared_head_smem(dim, vdim, same_kv) <= 227 * 1024) {
-#define SH_ARGS q, q_ld, q_hs, k, k_bs, k_ps, k_hs, v, v_bs, v_ps, v_hs, B, S, heads, kv_heads, dim, held, shift, pad, window, chunk, scale, softcap, sink, out, ld_out, out_col, dyn, ws, stream
+#define SH_ARGS q, q_ld, q_hs, k, k_bs, k_ps, k_hs, v, v_bs, v_ps, v_hs, B, S, heads, kv_heads, dim, held, shift, pad, window, chunk, scale, softcap, sink, out, ld_out, out_col, dyn, ws, back, back_interleaved, stream
         if (dtype == 1) return vdim == 128 ? launch_shared_head<__nv_bfloat16, 2>(SH_ARGS) : vdim == 256 ? launch_shared_head<__nv_bfloat16, 4>(SH_ARGS)
                                                                                                        : launch_shared_head<__nv_bfloat16, 8>(SH_ARGS);
         return vdim == 128 ? launch_shared_head<__half, 2>(SH_ARGS) : vdim == 256 ? launch_shared_head<__half, 4>(SH_ARGS)
@@ -928,7 +1049,7 @@ extern "C" int mixers_softmax_attention(int dtype, const void* q, long q_ld, lon
     long items = (long)B * S * heads;
     MIXERS_DISPATCH(dtype, softmax_attention_kernel<T><<<(unsigned)items, SA_WARPS * 32, smem, stream>>>(
         (const T*)q, q_ld, q_hs, (const T*)k, k_bs, k_ps, k_hs, (const T*)v, v_bs, v_ps, v_hs, B, S, heads, kv_heads, dim, vdim, held, shift, pad, window, chunk,
-        scale, softcap, (const T*)sink, (T*)out, ld_out, out_col, dyn, rows16 ? 1 : 0));
+        scale, softcap, (const T*)sink, (T*)out, ld_out, out_col, dyn, rows16 ? 1 : 0, back, back_interleaved));
     return mixers_status();
 }
 

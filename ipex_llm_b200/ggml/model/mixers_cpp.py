@@ -32,7 +32,11 @@ _SIGNATURES = {
                                                                  _c_ptr, _c_ptr],
     "mixers_gated_linear_attention": [_c_int, _c_ptr] + [_c_int] * 6 + [_c_ptr, _c_float, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_gated_rms_norm": [_c_int, _c_ptr, _c_long, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_float, _c_ptr, _c_int, _c_int,
-                              _c_float, _c_int, _c_ptr],
+                              _c_float, _c_int, _c_ptr, _c_ptr],
+    "mixers_mlstm": [_c_int, _c_ptr] + [_c_int] * 11 + [_c_ptr, _c_ptr, _c_float, _c_float, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
+                                                       _c_ptr],
+    "mixers_glu": [_c_int, _c_ptr, _c_long] + [_c_int] * 5 + [_c_ptr, _c_long, _c_ptr],
+    "mixers_rotary_table": [_c_ptr, _c_int, _c_float] + [_c_int] * 4 + [_c_ptr, _c_ptr, _c_ptr, _c_ptr],
     "mixers_short_conv": [_c_int, _c_ptr] + [_c_int] * 6 + [_c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_channel_delta_rule": [_c_int, _c_ptr] + [_c_int] * 6 + [_c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr,
                                                                    _c_ptr, _c_ptr],
@@ -42,9 +46,10 @@ _SIGNATURES = {
     "mixers_constant_decay_attention": [_c_int, _c_ptr] + [_c_int] * 7 + [_c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_rms_pair_sum": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_float, _c_long, _c_int, _c_ptr, _c_ptr],
     "mixers_sum_residual_norms": [_c_int, _c_ptr, _c_long, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_long, _c_int,
-                                  _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_long, _c_ptr],
+                                  _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_long, _c_float, _c_ptr],
     "mixers_gelu_erf": [_c_int, _c_ptr, _c_long, _c_ptr, _c_ptr],
-    "mixers_rope_qk_prepare": [_c_int, _c_ptr] + [_c_int] * 14 + [_c_ptr, _c_float, _c_ptr, _c_int, _c_float, _c_int, _c_ptr, _c_ptr, _c_long, _c_long,
+    "mixers_rope_qk_prepare": [_c_int, _c_ptr] + [_c_int] * 14 + [_c_ptr, _c_float, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_float, _c_ptr, _c_ptr,
+                                                                 _c_long, _c_long,
                                                                  _c_long, _c_ptr, _c_long, _c_long, _c_long, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_moe_scatter_scaled": [_c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_long, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "mixers_token_shift_mix": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr],
@@ -62,14 +67,14 @@ _SIGNATURES = {
                           _c_ptr, _c_ptr, _c_ptr, _c_ptr],
     "mixers_rms_residual": [_c_int, _c_ptr, _c_long, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_long, _c_int, _c_ptr, _c_ptr,
                             _c_ptr],
-    "mixers_rms_norm_rows": [_c_int, _c_ptr, _c_long, _c_int, _c_ptr, _c_ptr, _c_float, _c_ptr, _c_ptr],
+    "mixers_rms_norm_rows": [_c_int, _c_ptr, _c_long, _c_int, _c_ptr, _c_ptr, _c_float, _c_float, _c_ptr, _c_ptr],
     "mixers_xielu": [_c_int, _c_ptr, _c_long, _c_ptr, _c_ptr, _c_ptr],
     "mixers_silu_mul": [_c_int, _c_ptr, _c_long, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr],
     "mixers_gelu_table_mul": [_c_int, _c_ptr, _c_long, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_latent_prepare": [_c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr,
                               _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_softmax_attention": [_c_int, _c_ptr, _c_long, _c_long, _c_ptr, _c_long, _c_long, _c_long, _c_ptr, _c_long, _c_long, _c_long] + [_c_int] * 8
-                                + [_c_ptr, _c_int, _c_int, _c_float, _c_float, _c_ptr, _c_ptr, _c_long, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr],
+                                + [_c_ptr, _c_int, _c_int, _c_float, _c_float, _c_ptr, _c_ptr, _c_long, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr],
     "mixers_grouped_router": [_c_int, _c_ptr, _c_long, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr],
     "mixers_moe_small": [_c_int, _c_ptr, _c_long, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr,
                          _c_int, _c_int, _c_float, _c_float, _c_ptr, _c_ptr, _c_ptr, _c_ptr],

@@ -184,6 +184,11 @@ def _optimize_pre(model, qtype=None):
         import functools
         from ipex_llm_b200.transformers.models.bugipel import merge_projections
         model.apply(functools.partial(merge_projections, row_multiple=128 if qtype is not None else 0))
+    elif model_type == "rumuvik":
+        # everything that reads a mixer's input -> one in_proj, gate and up -> gate_up, mixer output and down projection -> one out_proj
+        import functools
+        from ipex_llm_b200.transformers.models.rumuvik import merge_projections
+        model.apply(functools.partial(merge_projections, row_multiple=128 if qtype is not None else 0))
     return model
 
 
@@ -215,7 +220,7 @@ def _optimize_post(model):
         convert_forward(model, module.MixtralRMSNorm, rms_norm_forward)
         convert_forward(model, module.MixtralModel, mixtral_model_forward)
         convert_forward(model, module.MixtralAttention, mixtral_attention_forward)
-    elif model_type in ("zafepel", "serotar", "zubedra", "nikedra", "bugipel"):
+    elif model_type in ("zafepel", "serotar", "zubedra", "nikedra", "bugipel", "rumuvik"):
         # this package's own model class: its forwards already call the fused operators and pick the state cache;
         # the recorded decode step for such a cache goes behind generate()
         from ipex_llm_b200.transformers.state_decode_graph import install_state_generate

@@ -469,7 +469,8 @@ class LatentKVLayer:
 
 
 class RecurrentStateLayer:
-    """What a linear recurrence carries from token to token: the matrix state [B, H, D, Dv] in 32-bit floats and, where a
+    """What a linear recurrence carries from token to token: the matrix state [B, H, D, Dv] in 32-bit floats (and, where it has them,
+    further 32-bit vectors) and, where a
     short convolution precedes it, the last ``taps - 1`` inputs of every channel [B, taps - 1, C].  Over several new tokens the
     convolution kernel reads ``tail`` and writes ``tail_next`` (no thread reads what another has replaced) and the caller copies
     it back; ``tail`` itself never moves.  A layer with more than one convolution (one on the mixer's input, another inside the
@@ -480,6 +481,14 @@ class RecurrentStateLayer:
         self.tail = None
         self.tail_next = None
         self.more_tails = {}              # key -> [tail, tail_next]
+        self.vectors = {}                 # key -> fp32 tensor [B, ...]
+
+    def vector(self, key, shape, device):
+        """what a recurrence carries beside its matrix (a normaliser, a running maximum): 32-bit, zeros before a sequence's first token"""
+        t = self.vectors.get(key)
+        if t is None:
+            t = self.vectors[key] = torch.zeros(shape, dtype=torch.float32, device=device)
+        return t
 
     def matrix(self, batch, heads, dim, vdim, device):
         if self.state is None:
@@ -499,7 +508,7 @@ class RecurrentStateLayer:
         return self.tail, self.tail_next
 
     def clear(self):
-        for t in [self.state, self.tail, self.tail_next] + [t for pair in self.more_tails.values() for t in pair]:
+        for t in [self.state, self.tail, self.tail_next] + [t for pair in self.more_tails.values() for t in pair] + list(self.vectors.values()):
             if t is not None:
                 t.zero_()
 
@@ -510,6 +519,7 @@ class RecurrentStateLayer:
                 setattr(self, name, t.index_select(0, index).contiguous())
         for pair in self.more_tails.values():
             pair[0], pair[1] = pair[0].index_select(0, index).contiguous(), pair[1].index_select(0, index).contiguous()
+        self.vectors = {k: t.index_select(0, index).contiguous() for k, t in self.vectors.items()}
 
 
 class MixerStateLayer:

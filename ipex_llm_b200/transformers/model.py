@@ -40,7 +40,8 @@ NATIVE_ARCHITECTURES = {"Zafepel": "ipex_llm_b200.transformers.models.zafepel",
                         "Serotar": "ipex_llm_b200.transformers.models.serotar",
                         "Zubedra": "ipex_llm_b200.transformers.models.zubedra",
                         "Nikedra": "ipex_llm_b200.transformers.models.nikedra",
-                        "Bugipel": "ipex_llm_b200.transformers.models.bugipel"}
+                        "Bugipel": "ipex_llm_b200.transformers.models.bugipel",
+                        "Rumuvik": "ipex_llm_b200.transformers.models.rumuvik"}
 
 
 def native_architecture(model_dir):

@@ -169,17 +169,35 @@ def constant_decay_attention(proj, off, heads, dim, vdim, decay, state, slot0, p
     return o
 
 
-def gated_rms_norm(o, gate, off_g, weight, eps, out, out_col, out_scale, sigmoid=False, gate_first=False):
+def mlstm(proj, off_q, off_k, off_v, off_i, off_f, heads, dim, vdim, bias_i, bias_f, cap, tiny, state, norm_state, max_state, slot0, pad):
+    """the mLSTM's matrix memory over the new tokens (q | k | v and the two gates' logits in columns of proj); state fp32
+    [B, heads, dim, vdim], norm_state fp32 [B, heads, dim] and max_state fp32 [B, heads, vdim + 1] in place; returns (o fp32
+    [B, S, heads, vdim], below fp32 [B, S, heads]): the read-out is o / below, which ``gated_rms_norm`` takes"""
+    B, S, P = proj.shape
+    states = ((state, (B, heads, dim, vdim)), (norm_state, (B, heads, dim)), (max_state, (B, heads, vdim + 1)))
+    invalidInputError(proj.is_contiguous() and max(off_q + heads * dim, off_k + heads * dim, off_v + heads * vdim, off_i + heads, off_f + heads) <= P
+                      and all(t.dtype == torch.float32 and t.is_contiguous() and t.shape == s for t, s in states)
+                      and all(t.numel() == heads and t.dtype == proj.dtype and t.is_contiguous() for t in (bias_i, bias_f)), "mlstm: unexpected layout")
+    o = torch.empty(B, S, heads, vdim, dtype=torch.float32, device=proj.device)
+    below = torch.empty(B, S, heads, dtype=torch.float32, device=proj.device)
+    native.call("mixers_mlstm", native.dtype_code(proj.dtype), native.ptr(proj), B, S, P, int(off_q), int(off_k), int(off_v), int(off_i), int(off_f), heads,
+                dim, vdim, native.ptr(bias_i), native.ptr(bias_f), float(cap), float(tiny), native.ptr(state), native.ptr(norm_state),
+                native.ptr(max_state), int(slot0), native.ptr(pad), native.ptr(o), native.ptr(below), native.stream(proj.device))
+    return o, below
+
+
+def gated_rms_norm(o, gate, off_g, weight, eps, out, out_col, out_scale, sigmoid=False, gate_first=False, below=None):
     """out[:, out_col:...] = out_scale * rms_norm(o per head) * weight * silu(gate columns from off_g); ``weight`` [vdim] serves
     every head, [heads * vdim] gives each head its own.  ``sigmoid``: the gate is sigmoid(.) instead of silu(.); ``gate_first``:
-    the gate multiplies before the norm (the root mean square is that of the gated values)"""
+    the gate multiplies before the norm (the root mean square is that of the gated values); ``below`` fp32 (one number per row and
+    head): o's heads are divided by it first"""
     heads, vdim = o.shape[-2], o.shape[-1]
     n = o.numel() // (heads * vdim)
     invalidInputError(o.is_contiguous() and o.dtype == torch.float32 and gate.is_contiguous() and out.is_contiguous() and out.shape[0] == n
-                      and gate.dtype == out.dtype and weight.numel() in (vdim, heads * vdim), "gated_rms_norm: unexpected layout")
+                      and (below is None or (below.dtype == torch.float32 and below.is_contiguous() and below.numel() == n * heads)) and gate.dtype == out.dtype and weight.numel() in (vdim, heads * vdim), "gated_rms_norm: unexpected layout")
     native.call("mixers_gated_rms_norm", native.dtype_code(out.dtype), native.ptr(o), n, heads, vdim, native.ptr(gate), gate.shape[-1], off_g,
                 native.ptr(weight), vdim if weight.numel() == heads * vdim and heads > 1 else 0, float(eps), native.ptr(out), out.shape[1], out_col,
-                float(out_scale), int(bool(sigmoid)) | (int(bool(gate_first)) << 1), native.stream(out.device))
+                float(out_scale), int(bool(sigmoid)) | (int(bool(gate_first)) << 1), native.ptr(below), native.stream(out.device))
 
 
 def token_shift_mix(h, mu, tail, tail_next, slot0, pad):
@@ -261,12 +279,13 @@ def rms_pair_sum(a, b, w_a, w_b, eps, scale):
 
 
 def sum_residual_norms(x, ys, out_dtype, eps, pre_gain=None, stack=None, index=0, coef=None, gain1=None, gain2=None, replace=False, vec=None,
-                       x_copy=None):
+                       x_copy=None, gain_add=0.0):
     """x += sum(ys) in place (x fp32 [N, W]; ``ys``: up to two tensors of the model's dtype and two fp32 ones); ``pre_gain``: x is
     first divided by its root mean square and multiplied by this scalar; with ``stack`` [streams, N, W] the new x is kept as
     stream ``index`` and, with ``coef`` [index + 1], replaced by the coefficient-weighted sum of streams 0..index.  ``replace``: the
     sum of ``ys`` takes x's place; ``vec`` [W] is added with them; ``x_copy`` [N, W] (a column range of a wider buffer) receives the
-    new x in ``out_dtype``.  Gains are one number or a vector [W].  Returns (x / rms(x) * gain1, x / rms(x) * gain2) in
+    new x in ``out_dtype``.  Gains are one number or a vector [W]; ``gain_add`` is added to them in 32-bit (1: weights stored around
+    zero).  Returns (x / rms(x) * gain1, x / rms(x) * gain2) in
     ``out_dtype`` (None where no gain is given)."""
     n, w = x.shape
     invalidInputError(x.dtype == torch.float32 and x.is_contiguous(), "sum_residual_norms: x is a contiguous fp32 [N, W]")
@@ -293,7 +312,8 @@ def sum_residual_norms(x, ys, out_dtype, eps, pre_gain=None, stack=None, index=0
     native.call("mixers_sum_residual_norms", native.dtype_code(out_dtype), native.ptr(x), n, w, native.ptr(typed[0]), native.ptr(typed[1]),
                 native.ptr(floats[0]), native.ptr(floats[1]), native.ptr(pre_gain), float(eps), native.ptr(stack), n * w, int(index),
                 native.ptr(coef), native.ptr(gain1), native.ptr(gain2), int(vectors), native.ptr(h1), native.ptr(h2), int(bool(replace)), native.ptr(vec),
-                native.ptr(x_copy), max(x_copy.stride(0), w) if x_copy is not None else w, native.stream(x.device))
+                native.ptr(x_copy), max(x_copy.stride(0), w) if x_copy is not None else w, float(gain_add),
+                native.stream(x.device))
     return h1, h2
 
 
@@ -305,22 +325,39 @@ def gelu_erf(z):
     return out
 
 
+def rotary_table(freq, amp, B, S, held, shift, pad, dyn=None):
+    """fp32 [B * S, pairs, 2]: cosine and sine (times ``amp``) of every new token's position * freq[i] (freq float64 [pairs])"""
+    invalidInputError(freq.dtype == torch.float64 and freq.is_contiguous(), "rotary_table: frequencies in double precision")
+    table = torch.empty(B * S, freq.numel(), 2, dtype=torch.float32, device=freq.device)
+    native.call("mixers_rotary_table", native.ptr(freq), freq.numel(), float(amp), B, S, int(held), int(shift), native.ptr(pad), native.ptr(dyn),
+                native.ptr(table), native.stream(freq.device))
+    return table
+
+
 def rope_qk_prepare(proj, off_q, off_k, off_v, heads, kv_heads, q_dim, k_dim, vdim, q_rot_off, k_rot_off, rot_dims, inv_freq, amp, k_store,
-                    k_strides, v_store, v_strides, held, shift, pad, eps=0.0, k_norm_w=None, k_norm_cols=0, dyn=None, unit_rms=False):
+                    k_strides, v_store, v_strides, held, shift, pad, eps=0.0, k_norm_w=None, k_norm_cols=0, dyn=None, unit_rms=False,
+                    table=None, v_table=None, interleaved=False, kv_proj=None):
     """rotary positions on the new tokens' queries and keys (columns of proj [B, S, P]) and the cache write of keys and values;
     ``k_strides`` / ``v_strides``: (batch, position, head) strides of the caches in elements; ``inv_freq`` float64 [rot_dims / 2],
     ``amp`` multiplies cosine and sine; ``k_norm_w``: the first ``k_norm_cols`` channels of every key head are RMS-normalised with
-    this weight; ``unit_rms``: behind the rotation every query and key head is divided by its root mean square.  Returns q
-    [B * S, heads * q_dim]"""
+    this weight; ``unit_rms``: behind the rotation every query and key head is divided by its root mean square.  ``table``
+    (``rotary_table``) replaces ``inv_freq`` and ``amp``; ``v_table`` rotates the values over all their channels; ``interleaved``: pairs
+    are channels (2i, 2i + 1); ``kv_proj`` [B, S, P2]: keys and values are columns of this buffer.  Returns q [B * S, heads * q_dim]"""
     B, S, P = proj.shape
+    for t, pairs in ((table, rot_dims // 2), (v_table, vdim // 2)):
+        invalidInputError(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == (B * S, pairs, 2)),
+                          "rope_qk_prepare: a table holds cosine and sine of every new token and pair")
+    invalidInputError(kv_proj is None or (kv_proj.is_contiguous() and kv_proj.shape[:2] == (B, S) and kv_proj.dtype == proj.dtype)
+                      and not (unit_rms and table is not None), "rope_qk_prepare: unexpected layout")
     invalidInputError(proj.is_contiguous() and k_store.dtype == proj.dtype and (v_store is None or v_store.dtype == proj.dtype)
-                      and (rot_dims == 0 or (inv_freq.dtype == torch.float64 and inv_freq.numel() == rot_dims // 2 and inv_freq.is_contiguous())),
+                      and (rot_dims == 0 or table is not None or (inv_freq.dtype == torch.float64 and inv_freq.numel() == rot_dims // 2 and inv_freq.is_contiguous())),
                       "rope_qk_prepare: unexpected layout")
     q = torch.empty(B * S, heads * q_dim, dtype=proj.dtype, device=proj.device)
     vs = v_strides if v_store is not None else (0, 0, 0)
     native.call("mixers_rope_qk_prepare", native.dtype_code(proj.dtype), native.ptr(proj), B, S, P, int(off_q), int(off_k), int(off_v), heads, kv_heads,
-                q_dim, k_dim, vdim if v_store is not None else 0, int(q_rot_off), int(k_rot_off), int(rot_dims), native.ptr(inv_freq) if rot_dims else None,
-                float(amp), native.ptr(k_norm_w), int(k_norm_cols), float(eps), int(bool(unit_rms)), native.ptr(q), native.ptr(k_store), *[int(v) for v in k_strides],
+                q_dim, k_dim, vdim if v_store is not None else 0, int(q_rot_off), int(k_rot_off), int(rot_dims), native.ptr(inv_freq) if rot_dims and table is None else None,
+                float(amp), native.ptr(table), native.ptr(v_table), int(bool(unit_rms)) | (int(bool(interleaved)) << 1), native.ptr(kv_proj),
+                kv_proj.shape[-1] if kv_proj is not None else 0, native.ptr(k_norm_w), int(k_norm_cols), float(eps), native.ptr(q), native.ptr(k_store), *[int(v) for v in k_strides],
                 native.ptr(v_store), *[int(v) for v in vs], int(held), int(shift), native.ptr(pad), native.ptr(dyn), native.stream(proj.device))
     return q
 
@@ -375,11 +412,12 @@ def rms_residual(x, y, gain, vec, eps, out_dtype, stack=None, index=0, coef=None
     return h
 
 
-def rms_norm_rows(x, gain, vec, eps, out_dtype):
+def rms_norm_rows(x, gain, vec, eps, out_dtype, vec_add=0.0):
+    """x / rms(x) * gain * (vec_add + vec) in ``out_dtype`` (x fp32; ``gain`` one number, ``vec`` [W], either may be None)"""
     x = _c(x)
     out = torch.empty(x.shape, dtype=out_dtype, device=x.device)
     native.call("mixers_rms_norm_rows", native.dtype_code(out_dtype), native.ptr(x), x.numel() // x.shape[-1], x.shape[-1], native.ptr(gain),
-                native.ptr(vec), float(eps), native.ptr(out), native.stream(x.device))
+                native.ptr(vec), float(vec_add), float(eps), native.ptr(out), native.stream(x.device))
     return out
 
 
@@ -401,12 +439,37 @@ def silu_mul(gate_up, cols):
     return out
 
 
+def gelu_tanh_mul(gate_up, cols, out=None):
+    """gelu_tanh(first ``cols`` columns) * the next ``cols`` columns; ``out``: a column range of a contiguous buffer that receives it"""
+    gate_up = _c(gate_up)
+    n = gate_up.numel() // gate_up.shape[-1]
+    if out is None:
+        out = torch.empty(n, cols, dtype=gate_up.dtype, device=gate_up.device)
+    invalidInputError(out.shape == (n, cols) and out.dtype == gate_up.dtype and out.stride(1) == 1 and 2 * cols <= gate_up.shape[-1],
+                      "gelu_tanh_mul: unexpected layout")
+    if n:
+        native.call("mixers_glu", native.dtype_code(gate_up.dtype), native.ptr(gate_up), n, gate_up.shape[-1], 0, cols, cols, 1, native.ptr(out),
+                    max(out.stride(0), cols), native.stream(out.device))
+    return out
+
+
 def gelu_table_mul(g, table, col0, ids):
     """gelu_tanh(g [N, C]) * table[ids, col0 : col0 + C]"""
     g, ids = _c(g), _c(ids)
     out = torch.empty_like(g)
     native.call("mixers_gelu_table_mul", native.dtype_code(g.dtype), native.ptr(g), g.shape[0], g.shape[1], native.ptr(table), table.shape[1], int(col0),
                 native.ptr(ids), native.ptr(out), native.stream(g.device))
+    return out
+
+
+def rms_norm_columns(proj, off, cols, w, eps, held, shift, pad, dyn=None):
+    """[B * S, cols]: the columns off .. off + cols - 1 of proj [B, S, P], each row's divided by their root mean square and multiplied by
+    ``w`` (zeros for padding)"""
+    B, S, P = proj.shape
+    invalidInputError(proj.is_contiguous() and off + cols <= P and w.numel() == cols and w.dtype == proj.dtype, "rms_norm_columns: unexpected layout")
+    out = torch.empty(B * S, cols, dtype=proj.dtype, device=proj.device)
+    native.call("mixers_latent_prepare", native.dtype_code(proj.dtype), native.ptr(proj), B, S, P, int(off), cols, native.ptr(w), 0, 0, None, float(eps),
+                native.ptr(out), None, 0, int(held), int(shift), native.ptr(pad), native.ptr(dyn), native.stream(proj.device))
     return out
 
 
@@ -423,17 +486,20 @@ def latent_prepare(proj, off_q, q_rank, q_w, off_c, kv_rank, c_w, eps, store, he
 
 
 def softmax_attention(q, k, v, B, S, heads, held, shift, pad, window, scale, out=None, out_col=0, dyn=None, tensor_cores=True, softcap=0.0,
-                      sink=None, chunk=0):
+                      sink=None, chunk=0, back=None, back_interleaved=False):
     """q [B * S, heads * dim], or [B * S, heads, dim] with any token and head strides; k [B, L, kv_heads, dim], v [B, L, kv_heads,
     vdim] views (any strides with a unit last one); returns out [B * S, heads * vdim] in q's dtype.  ``softcap`` > 0 caps the
     scaled scores (cap * tanh(score / cap)); ``sink`` [heads]: a per-head term exp(sink) in the softmax's denominator;
-    ``chunk`` > 0: a query sees only the earlier positions of its own chunk of that many positions"""
+    ``chunk`` > 0: a query sees only the earlier positions of its own chunk of that many positions; ``back`` (a ``rotary_table`` of
+    vdim / 2 pairs): every head's output is turned back by its angles (``back_interleaved``: pairs are channels (2i, 2i + 1))"""
     kv_heads, dim, vdim = k.shape[2], k.shape[3], v.shape[3]
     q_hs = q.stride(1) if q.dim() == 3 else dim
     invalidInputError(q.stride(-1) == 1 and k.stride(-1) == 1 and v.stride(-1) == 1 and q.numel() == B * S * heads * dim and k.dtype == q.dtype
                       and v.dtype == q.dtype and v.shape[2] == kv_heads and (dyn is not None or (k.shape[1] >= held + S and v.shape[1] >= held + S)),
                       "softmax_attention: unexpected layout")
     invalidInputError(sink is None or (sink.numel() == heads and sink.dtype == q.dtype and sink.is_contiguous()), "softmax_attention: one sink per head")
+    invalidInputError(back is None or (back.dtype == torch.float32 and back.is_contiguous() and back.shape == (B * S, vdim // 2, 2) and vdim % 2 == 0),
+                      "softmax_attention: the table of angles holds cosine and sine of every new token and pair")
     if out is None:
         out = torch.empty(B * S, heads * vdim, dtype=q.dtype, device=q.device)
     need = native.lib().mixers_softmax_attention_workspace(native.dtype_code(q.dtype), B, S, heads, kv_heads, dim, vdim) if tensor_cores else 0
@@ -442,7 +508,7 @@ def softmax_attention(q, k, v, B, S, heads, held, shift, pad, window, scale, out
                 k.stride(2), native.ptr(v), v.stride(0), v.stride(1), v.stride(2), B, S, heads, kv_heads, dim, vdim, int(held), int(shift),
                 native.ptr(pad), int(window), int(chunk), float(scale), float(softcap or 0.0), native.ptr(sink), native.ptr(out), out.stride(0), int(out_col),
                 native.ptr(dyn), int(bool(tensor_cores)),
-                native.ptr(ws), native.stream(q.device))
+                native.ptr(ws), native.ptr(back), int(bool(back_interleaved)), native.stream(q.device))
     return out
 
 

@@ -1,7 +1,8 @@
 """Pieces that several of this package's own designs are built from: the rotary frequencies of a ``rot`` block, a lone weight under
 a module of its own, short convolutions on a layer's state, and the **delta rule with a decay per key channel** (behind short
-convolutions, unit-norm q / k, a per-head RMS norm of the read-out and a low-rank sigmoid gate) with its module tree.  The
-kernels are those of ``mixer_ops``."""
+convolutions, unit-norm q / k, a per-head RMS norm of the read-out and a low-rank sigmoid gate) with its module tree, and the
+attention over a **latent cache** whose rows hold a normalised latent and one rotated key part that all heads share.  The kernels
+are those of ``mixer_ops``."""
 import math
 
 import torch
@@ -10,6 +11,7 @@ from torch import nn
 from ipex_llm_b200.transformers.models import mixer_ops as ops
 from ipex_llm_b200.utils.common import invalidInputError
 
+ABSORB_MAX_TOKENS = 16        # up to this many new tokens per row attend to a latent cache itself (no key / value expansion)
 YARN_AMP_SLOPE = 0.1          # cosine and sine of rescaled frequencies are multiplied by slope * ln(factor) + 1
 
 
@@ -52,6 +54,59 @@ class Rotary:
         if t is None:
             t = self._on[device] = torch.tensor(self.freq or [0.0], dtype=torch.float64).to(device)
         return t
+
+
+class Angles:
+    """cosine and sine of every new token and rotated pair, formed once per call for all layer runs that share the frequencies"""
+
+    def __init__(self, B, S, cache, dyn):
+        self.B, self.S, self.cache, self.dyn = B, S, cache, dyn
+        self._tables = {}
+
+    def of(self, rotary, device):
+        """fp32 [B * S, pairs, 2], or None where nothing is rotated"""
+        if not rotary.freq:
+            return None
+        key = (tuple(rotary.freq), rotary.amp)
+        t = self._tables.get(key)
+        if t is None:                                        # position = slot - padding; a recorded step reads its slot from the device
+            t = self._tables[key] = ops.rotary_table(rotary.inv_freq(device), rotary.amp, self.B, self.S, self.cache.seen, 0, self.cache.pad, dyn=self.dyn)
+        return t
+
+
+def latent_expansion(uk, uv, heads, dim, rot_dim, vdim, rank):
+    """[heads * (dim + rot_dim) + heads * vdim, rank + rot_dim] from per-head key rows uk [heads * dim, rank] and value rows uv
+    [heads * vdim, rank]: turns cache rows [latent | rotated key part] into every head's key [W_uk latent | rotated part] and value
+    W_uv latent; per head the key rows are (W_uk_h 0; 0 I), the value rows (W_uv_h 0)"""
+    keys = torch.zeros(heads, dim + rot_dim, rank + rot_dim, dtype=uk.dtype)
+    keys[:, :dim, :rank] = uk.view(heads, dim, rank)
+    keys[:, dim:, rank:] = torch.eye(rot_dim, dtype=uk.dtype)
+    values = torch.zeros(heads * vdim, rank + rot_dim, dtype=uk.dtype)
+    values[:, :rank] = uv
+    return torch.cat([keys.view(heads * (dim + rot_dim), rank + rot_dim), values], dim=0)
+
+
+def latent_cache_attention(q, w, store, B, S, heads, q_dim, vdim, rank, held, shift, pad, scale, out, window=0, dyn=None, tensor_cores=True):
+    """out[:, : heads * vdim] = softmax attention of the new tokens' queries q [B * S, heads * q_dim] over the cache rows ``store`` [B,
+    capacity, rank + rotated part]; ``w``: ``latent_expansion``.
+
+    Few new tokens move their queries into the cache rows' space (W_uk_h^T q | rotated q): the cache itself is then the key of one
+    shared head, its latent part the value, and W_uv_h maps the weighted latents back.  A prompt or a long portion expands the keys
+    and values of the positions that some new token still sees."""
+    H, N, row = heads, B * S, store.shape[2]
+    if S <= ABSORB_MAX_TOKENS:
+        wk, wv = w[:H * q_dim].view(H, q_dim, row), w[H * q_dim:].view(H, vdim, row)[:, :, :rank]
+        qa = torch.matmul(q.view(N, H, q_dim).transpose(0, 1), wk).transpose(0, 1)                  # [N, H, row], stored head by head
+        rows = store.unsqueeze(2)                                            # [B, capacity, 1, row]
+        o_rows = ops.softmax_attention(qa, rows, rows[..., :rank], B, S, H, held, shift, pad, window, scale, dyn=dyn)
+        o = torch.matmul(o_rows.view(N, H, rank).transpose(0, 1), wv.transpose(1, 2))               # [H, N, vdim]
+        out[:, :H * vdim].unflatten(1, (H, vdim)).copy_(o.transpose(0, 1))
+        return
+    first = max(held - (window - 1), 0) if window > 0 else 0
+    total = held + S
+    kvx = torch.nn.functional.linear(store[:, first:total], w)               # [B, total - first, H * (q_dim + vdim)]
+    k, v = kvx[..., :H * q_dim].view(B, total - first, H, q_dim), kvx[..., H * q_dim:].view(B, total - first, H, vdim)
+    ops.softmax_attention(q, k, v, B, S, H, held - first, shift + first, pad, window, scale, out=out, tensor_cores=tensor_cores)
 
 
 class Weight(nn.Module):

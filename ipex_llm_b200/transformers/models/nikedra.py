@@ -36,12 +36,11 @@ from transformers.modeling_outputs import CausalLMOutputWithPast
 from ipex_llm_b200.transformers.kv import DynamicStateCache
 from ipex_llm_b200.transformers.models import experts, mixer_ops as ops
 from ipex_llm_b200.transformers.models.common import merge_linear
-from ipex_llm_b200.transformers.models.mixers import (ChannelDeltaMixer, Rotary, Weight, channel_delta, plain_linears, rotary_frequencies,  # noqa: F401
-                                                      short_conv)
+from ipex_llm_b200.transformers.models.mixers import (ABSORB_MAX_TOKENS, ChannelDeltaMixer, Rotary, Weight, channel_delta,  # noqa: F401
+                                                      latent_cache_attention, latent_expansion, plain_linears, rotary_frequencies, short_conv)
 from ipex_llm_b200.transformers.models.utils import read_safetensors
 from ipex_llm_b200.utils.common import invalidInputError
 
-ABSORB_MAX_TOKENS = 16        # up to this many new tokens per row attend to the latent cache itself (no key / value expansion)
 OVERLAP_MIN_TOKENS = 256      # from this many new tokens on, a layer's feed-forward runs on a second stream beside its mixer
 
 
@@ -97,13 +96,7 @@ class LatentRopeAttention(nn.Module):
 
     def expansion(self, uk, uv):
         """``expand`` from the checkpoint's per-head key rows uk [heads * dim, kv_rank] and value rows uv [heads * vdim, kv_rank]"""
-        H, D, Dr, Dv, R = self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank
-        keys = torch.zeros(H, D + Dr, R + Dr, dtype=uk.dtype)
-        keys[:, :D, :R] = uk.view(H, D, R)
-        keys[:, D:, R:] = torch.eye(Dr, dtype=uk.dtype)
-        values = torch.zeros(H * Dv, R + Dr, dtype=uk.dtype)
-        values[:, :R] = uv
-        return torch.cat([keys.view(H * (D + Dr), R + Dr), values], dim=0)
+        return latent_expansion(uk, uv, self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank)
 
 
 class ChunkedAttention(nn.Module):
@@ -285,25 +278,9 @@ class NikedraForCausalLM(PreTrainedModel, GenerationMixin):
                                 store, (cap * Rk, Rk, 0), None, None, held, shift, cache.pad, eps=self.config.norm_eps,
                                 k_norm_w=mx.dkv_norm.weight, k_norm_cols=R, dyn=dyn)
         kv.commit(S)
-        w = mx.expand.weight
-        if S <= ABSORB_MAX_TOKENS:
-            # few new tokens: the query of head h moves into the cache rows' space (W_uk_h^T q | rotated q), the cache itself is
-            # the key of one shared head, its latent part (the first R numbers of a row) the value, and W_uv_h maps the weighted
-            # latents back
-            wk, wv = w[:H * Dq].view(H, Dq, Rk), w[H * Dq:].view(H, Dv, Rk)[:, :, :R]
-            qa = torch.matmul(q.view(N, H, Dq).transpose(0, 1), wk).transpose(0, 1)                  # [N, H, Rk], stored head by head
-            rows = store.unsqueeze(2)                                        # [B, capacity, 1, Rk]
-            o_rows = ops.softmax_attention(qa, rows, rows[..., :R], B, S, H, held, shift, cache.pad, mx.window, mx.scale, dyn=dyn)
-            o = torch.matmul(o_rows.view(N, H, R).transpose(0, 1), wv.transpose(1, 2)).transpose(0, 1).reshape(N, H * Dv)
-        else:
-            # a prompt or a long portion: keys and values of the positions that some new token still sees, expanded from the cache
-            first = max(held - (mx.window - 1), 0)
-            total = held + S
-            kvx = torch.nn.functional.linear(store[:, first:total], w)      # [B, total - first, H * (Dq + Dv)]
-            k = kvx[..., :H * Dq].view(B, total - first, H, Dq)
-            v = kvx[..., H * Dq:].view(B, total - first, H, Dv)
-            o = ops.softmax_attention(q, k, v, B, S, H, held - first, shift + first, cache.pad, mx.window, mx.scale,
-                                      tensor_cores=self.attention_tensor_cores)
+        o = torch.empty(N, H * Dv, dtype=h.dtype, device=h.device)
+        latent_cache_attention(q, mx.expand.weight, store, B, S, H, Dq, Dv, R, held, shift, cache.pad, mx.scale, o, window=mx.window, dyn=dyn,
+                               tensor_cores=self.attention_tensor_cores)
         ops.sigmoid_gate(o, proj, off_g, 1)
         return mx.o_proj(o)
 
