@@ -687,12 +687,12 @@ def main():
     ap.add_argument("--no-prefill", action="store_true")
     ap.add_argument("--no-tp", action="store_true")
     ap.add_argument("--fused-mlp", type=int, default=1, dest="fused_mlp")
-    ap.add_argument("--arch", default="llama", choices=["llama", "zafepel", "serotar", "zubedra", "nikedra", "bugipel"],
-                    help="llama: the headline workload (default, unchanged); zafepel / serotar / zubedra / nikedra / bugipel: that design at real layer sizes "
-                         "beside the closest model of equal size (a Llama / a Mixtral / a Serotar / a Serotar / a Zafepel), with every kernel of the design "
-                         "against its roofline (bench_mixers.py / bench_serotar.py / bench_zubedra.py / bench_nikedra.py / bench_bugipel.py)")
-    ap.add_argument("--no-compare", action="store_true", help="--arch zafepel / serotar / zubedra / nikedra / bugipel: leave out the model of equal size")
-    ap.add_argument("--sizes", default=None, help="--arch nikedra / bugipel: only these of its sets of layer sizes (comma-separated, e.g. 2048)")
+    ap.add_argument("--arch", default="llama", choices=["llama", "zafepel", "serotar", "zubedra", "nikedra", "bugipel", "rumuvik"],
+                    help="llama: the headline workload (default, unchanged); zafepel / serotar / zubedra / nikedra / bugipel / rumuvik: that design at real layer sizes "
+                         "beside the closest model of equal size (a Llama / a Mixtral / a Serotar / a Serotar / a Zafepel / a Nikedra), with every kernel of the design "
+                         "against its roofline (bench_mixers.py / bench_serotar.py / bench_zubedra.py / bench_nikedra.py / bench_bugipel.py / bench_rumuvik.py)")
+    ap.add_argument("--no-compare", action="store_true", help="--arch zafepel / serotar / zubedra / nikedra / bugipel / rumuvik: leave out the model of equal size")
+    ap.add_argument("--sizes", default=None, help="--arch nikedra / bugipel / rumuvik: only these of its sets of layer sizes (comma-separated, e.g. 2048)")
     args = ap.parse_args()
     if args.arch == "zafepel":
         import bench_mixers
@@ -713,6 +713,10 @@ def main():
     if args.arch == "bugipel":
         import bench_bugipel
         bench_bugipel.run(args)
+        return
+    if args.arch == "rumuvik":
+        import bench_rumuvik
+        bench_rumuvik.run(args)
         return
     global FUSED_MLP
     FUSED_MLP = bool(args.fused_mlp)

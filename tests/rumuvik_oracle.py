@@ -127,20 +127,26 @@ def mlstm_gates(i_logit, f_logit, cap):
     return i, torch.nn.functional.logsigmoid(z)
 
 
-def mlstm_scan(q, k, v, i, f, state=None):
-    """q (already scaled), k [T, H, D]; v [T, H, Dv]; i, f [T, H] log gates.  Returns (outputs [T, H, Dv], (S, n, m))"""
+def mlstm_parts(q, k, v, i, f, state=None):
+    """q (already scaled), k [T, H, D]; v [T, H, Dv]; i, f [T, H] log gates.  Returns (S^T q [T, H, Dv], denominators [T, H], (S, n, m))"""
     T, H, D = q.shape
     S, n, m = state if state is not None else (torch.zeros(H, D, v.shape[-1], dtype=q.dtype), torch.zeros(H, D, dtype=q.dtype), torch.zeros(H, dtype=q.dtype))
-    out = []
+    above, below = [], []
     for t in range(T):
         new = torch.maximum(f[t] + m, i[t])
         keep, take = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
         m = new
         S = keep[:, None, None] * S + take[:, None, None] * k[t].unsqueeze(-1) * v[t].unsqueeze(-2)
         n = keep[:, None] * n + take[:, None] * k[t]
-        below = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
-        out.append(torch.einsum("hij,hi->hj", S, q[t]) / below[:, None])
-    return torch.stack(out), (S, n, m)
+        below.append(torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6)
+        above.append(torch.einsum("hij,hi->hj", S, q[t]))
+    return torch.stack(above), torch.stack(below), (S, n, m)
+
+
+def mlstm_scan(q, k, v, i, f, state=None):
+    """(outputs [T, H, Dv], (S, n, m))"""
+    above, below, state = mlstm_parts(q, k, v, i, f, state)
+    return above / below.unsqueeze(-1), state
 
 
 def mlstm_mixer(h, W, m, eps):
@@ -198,3 +204,65 @@ def greedy(cfg, weights, prompt, n_new):
     for _ in range(n_new):
         tokens.append(int(forward(cfg, weights, tokens)[-1].argmax()))
     return tokens
+
+
+# ------------------------------------------------------------------ random models
+ATT = dict(heads=6, kv_heads=2, dim=12, vdim=10, rot_dims=8, base=50.0, scale=0.5, softcap=4.0)
+LAT = dict(heads=4, dim=10, rot_dim=6, vdim=14, kv_rank=18, q_rank=22, base=300.0, scale=0.4, scaling=dict(factor=3.0, original=64, fast=8.0, slow=1.0))
+MEM = dict(heads=3, dim=10, vdim=14, gate_cap=6.0)
+
+
+def random_config(width=40, vocab=61, order=("attention", "latent_attention", "mlstm", "attention"), ffs=(24, 56, None, 33), att=None, lat=None, mem=None,
+                  loop=(1, 3, 3), eps=1e-5, embed_scale=2.5):
+    """``order``: the layers' mixers; ``ffs``: per layer the feed-forward's width or None; the dicts override the sizes above;
+    ``loop``: (start, stop, times) or None"""
+    a, l, m = (dict(base, **(over or {})) for base, over in ((ATT, att), (LAT, lat), (MEM, mem)))
+    rot_l = {"base": l["base"], "dims": l["rot_dim"]}
+    if l["scaling"]:
+        rot_l["scaling"] = dict(l["scaling"])
+    mixers = {"attention": dict({k: a[k] for k in ("heads", "kv_heads", "dim", "vdim", "scale", "softcap")}, rot={"base": a["base"], "dims": a["rot_dims"]}),
+              "latent_attention": dict({k: l[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank", "scale")}, rot=rot_l),
+              "mlstm": dict(m)}
+    layers = [{"type": kind, "mixer": mixers[kind], "mlp": None if ff is None else {"kind": "dense", "ff": ff}} for kind, ff in zip(order, ffs)]
+    cfg = {"architecture": "Rumuvik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "embedding": {"scale": embed_scale}, "layers": layers}
+    if loop:
+        cfg["loop"] = {"start": loop[0], "stop": loop[1], "times": loop[2]}
+    return cfg
+
+
+def random_weights(cfg, seed, dtype=torch.bfloat16):
+    """weights under the checkpoint's names"""
+    g = torch.Generator().manual_seed(seed)
+    W = cfg["width"]
+
+    def mat(o, i, s=1.0):
+        return torch.randn(o, i, generator=g) * (s / math.sqrt(i))
+
+    def vec(n, mean=0.0, s=0.2):
+        return mean + torch.randn(n, generator=g) * s
+
+    w = {"embed": torch.randn(cfg["vocab"], W, generator=g), "final.norm": vec(W), "head": mat(cfg["vocab"], W)}
+    for i, lc in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", lc["mixer"]
+        w[p + "norm1"] = vec(W)
+        x = p + "mix."
+        H, D, Dv = m["heads"], m["dim"], m["vdim"]
+        if lc["type"] == "attention":
+            G = m["kv_heads"]
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * Dv)):
+                w[x + n], w[x + n + ".b"] = mat(rows, W, 1.5), vec(rows, 0.0, 0.5)
+        elif lc["type"] == "latent_attention":
+            R, Dr, Q = m["kv_rank"], m["rot_dim"], m["q_rank"]
+            w[x + "dq"], w[x + "dq.norm"], w[x + "uq"] = mat(Q, W), vec(Q, 1.0), mat(H * (D + Dr), Q, 1.5)
+            w[x + "dkv"], w[x + "dkv.norm"] = mat(R + Dr, W, 1.5), vec(R, 1.0)
+            w[x + "uk"], w[x + "uv"] = mat(H * D, R, 1.5), mat(H * Dv, R)
+        else:
+            for n, rows in (("q", H * D), ("k", H * D), ("v", H * Dv), ("g", H * Dv)):
+                w[x + n] = mat(rows, W, 1.5)
+            w[x + "i"], w[x + "f"] = mat(H, W, 2.0), mat(H, W, 1.5)
+            w[x + "i.b"], w[x + "f.b"], w[x + "norm"] = vec(H, -0.5, 1.0), vec(H, 2.5, 1.0), vec(H * Dv, 1.0)
+        w[x + "o"] = mat(W, H * Dv)
+        if lc.get("mlp") is not None:
+            F = lc["mlp"]["ff"]
+            w[p + "norm2"], w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"] = vec(W), mat(F, W, 2.0), mat(F, W), mat(W, F)
+    return {k: v.to(dtype) for k, v in w.items()}
